@@ -6,6 +6,7 @@ from .vekedra import VekedraConfig
 from .figotar import FigotarConfig
 from .vatevik import VatevikConfig
 from .divitar import DivitarConfig
+from .fororax import FororaxConfig
 
 for _name in ("GPT2LMHeadModel", "TinyGPT", "gpt2"):
     register_architecture(_name, GPT2Config)
@@ -13,6 +14,7 @@ register_architecture("Vekedra", VekedraConfig)
 register_architecture("Figotar", FigotarConfig)
 register_architecture("Vatevik", VatevikConfig)
 register_architecture("Divitar", DivitarConfig)
+register_architecture("Fororax", FororaxConfig)
 
-__all__ = ["ConfigError", "LayerSpec", "ModelSpec", "PartSpec", "GPT2Config", "VekedraConfig", "FigotarConfig", "VatevikConfig", "DivitarConfig", "architecture_name",
+__all__ = ["ConfigError", "LayerSpec", "ModelSpec", "PartSpec", "GPT2Config", "VekedraConfig", "FigotarConfig", "VatevikConfig", "DivitarConfig", "FororaxConfig", "architecture_name",
            "config_from_dict", "known_architectures", "load_config", "register_architecture"]

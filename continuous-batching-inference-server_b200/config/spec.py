@@ -47,6 +47,8 @@ class LayerSpec:
     # a constant on everything the layer adds to the stream (1: none), and a third part after the feed-forward that
     # reads the stream as it is (a feed-forward kind; None: the layer has none); for the arrangements that know them
     residual_scale: float = 1.0
+    # a constant on the stream before a part's result joins it (1: none), for the arrangements that know it
+    stream_scale: float = 1.0
     side: Optional[PartSpec] = None
 
 

@@ -17,7 +17,8 @@
 // The lane-group form also takes values of another width than the keys (hdv; lane i of a group holds entries
 // 8i .. 8i+7 of both), values that are the first entries of the keys' rows (vc == kc, v_row: elements between two
 // tokens' values), a distance bias (slope[h] * (p - j) taken off the score), a query temperature by position and a
-// sink in the denominator.
+// sink in the denominator.  The bias may grow with the logarithm of the distance instead (rates), and with v_heads > 1
+// every query head attends to the values of every key/value head (head_place in common.cuh).
 #include "attention_decode_tc.cuh"
 #include <math.h>
 
@@ -35,7 +36,8 @@ paged_decode_bf16_kernel(const __nv_bfloat16* qkv, int ld, int k_off, int v_off,
                          __nv_bfloat16* __restrict__ out, int out_ld, float* part,
                          unsigned int* counters, int n_head, int n_kv_head, int hd, int ps, float scale,
                          int window, int nsplit, int hdv, int v_row, const float* __restrict__ slopes,
-                         const float* __restrict__ sinks, float temp_coef, int temp_every) {
+                         const float* __restrict__ sinks, float temp_coef, int temp_every, const float* __restrict__ rates,
+                         int v_heads) {
   constexpr int G = 32 / LPK;             // key groups per warp
   constexpr int NW = DEC_WARPS * G;       // key workers per block
   __shared__ float sm_m[DEC_WARPS], sm_l[DEC_WARPS];
@@ -51,7 +53,8 @@ paged_decode_bf16_kernel(const __nv_bfloat16* qkv, int ld, int k_off, int v_off,
       for (int t = threadIdx.x; t < hdv; t += blockDim.x) out[(size_t)row * out_ld + h * hdv + t] = __float2bfloat16_rn(0.f);
     return;
   }
-  const int hk = h / (n_head / n_kv_head);
+  const HeadPlace hp = head_place(h, n_head, n_kv_head, v_heads);
+  const int hk = hp.key, hv = hp.value;
   const int pos = positions[row];
   const int kend = pos + 1;
   const int kstart = first_seen(pos, window);
@@ -64,11 +67,12 @@ paged_decode_bf16_kernel(const __nv_bfloat16* qkv, int ld, int k_off, int v_off,
   const bool fused = k_off >= 0;
   if (temp_every > 0) scale *= 1.0f + temp_coef * logf((float)((pos + 1) / temp_every + 1));
   const float slope = slopes ? slopes[h] : 0.f;
+  const float* rate = rates ? rates + h : nullptr;
 
   float q[8];
   {
     uint4 raw = make_uint4(0, 0, 0, 0);
-    if (active) raw = *reinterpret_cast<const uint4*>(qkv + (size_t)row * ld + h * hd + sub * 8);
+    if (active) raw = *reinterpret_cast<const uint4*>(qkv + (size_t)row * ld + hp.query * hd + sub * 8);
     unpack8(raw, q);
 #pragma unroll
     for (int i = 0; i < 8; ++i) q[i] *= scale;
@@ -89,18 +93,20 @@ paged_decode_bf16_kernel(const __nv_bfloat16* qkv, int ld, int k_off, int v_off,
       if (j < ke && (active || active_v)) {
         if (fused && j == pos) {
           if (active) kk[u] = *reinterpret_cast<const uint4*>(qkv + (size_t)row * ld + k_off + hk * hd + sub * 8);
-          if (active_v) vv[u] = *reinterpret_cast<const uint4*>(qkv + (size_t)row * ld + v_off + hk * hdv + sub * 8);
+          if (active_v) vv[u] = *reinterpret_cast<const uint4*>(qkv + (size_t)row * ld + v_off + hv * hdv + sub * 8);
           const int slot = slot_mapping[row];
           if (slot >= 0) {
             const size_t token = ((size_t)(slot / ps) * n_kv_head + hk) * ps + (slot % ps);
+            const size_t v_token = ((size_t)(slot / ps) * n_kv_head + hv) * ps + (slot % ps);
             if (active) *reinterpret_cast<uint4*>(kc + token * hd + sub * 8) = kk[u];
-            if (active_v && vc != kc) *reinterpret_cast<uint4*>(vc + token * v_row + sub * 8) = vv[u];
+            if (active_v && vc != kc) *reinterpret_cast<uint4*>(vc + v_token * v_row + sub * 8) = vv[u];
           }
         } else {
           const int page = bt[j / ps];
           const size_t token = ((size_t)page * n_kv_head + hk) * ps + (j % ps);
           if (active) kk[u] = *reinterpret_cast<const uint4*>(kc + token * hd + sub * 8);
-          if (active_v) vv[u] = *reinterpret_cast<const uint4*>(vc + token * v_row + sub * 8);
+          const size_t v_token = ((size_t)page * n_kv_head + hv) * ps + (j % ps);
+          if (active_v) vv[u] = *reinterpret_cast<const uint4*>(vc + v_token * v_row + sub * 8);
         }
       }
     }
@@ -126,7 +132,7 @@ paged_decode_bf16_kernel(const __nv_bfloat16* qkv, int ld, int k_off, int v_off,
       for (int i = 0; i < 8; ++i) d = fmaf(q[i], kf[i], d);
 #pragma unroll
       for (int o = LPK / 2; o > 0; o >>= 1) d += __shfl_xor_sync(0xffffffffu, d, o);
-      s[u] = valid[u] ? d - slope * (float)(pos - (base + u * NW + wkr)) : -INFINITY;
+      s[u] = valid[u] ? (slope != 0.f ? d - distance_bias(slope, rate, (float)(pos - (base + u * NW + wkr))) : d) : -INFINITY;
     }
     float m_new = m;
 #pragma unroll
@@ -303,15 +309,16 @@ CBIS_EXPORT int cbis_paged_decode_bf16(const void* qkv, int ld, int k_off, int v
                                        float* part, unsigned int* counters, int rows, int n_head, int n_kv_head,
                                        int hd, int ps, float scale, int window, int nsplit, void* stream, int hdv,
                                        int v_row, const float* slopes, const float* sinks, float temp_coef,
-                                       int temp_every) {
+                                       int temp_every, const float* rates, int v_heads) {
   if (rows <= 0) return CBIS_OK;
   // hdv (0: the keys' width, values in pages of their own): the values' width.  With values of another width or in
   // the keys' rows, a bias or a temperature the lane-group form runs whatever the head size; a sink alone is
   // taken by both forms (it joins the denominator where the parts are merged)
   if (hdv <= 0) hdv = hd, v_row = hd;
-  const bool extended = hdv != hd || v_row != hd || slopes || temp_every > 0;
+  const bool extended = hdv != hd || v_row != hd || slopes || temp_every > 0 || v_heads > 1;
+  if (v_heads != 1 && (v_heads != n_kv_head || n_head % v_heads)) return CBIS_ERR_BAD_SIZE;
   if (hdv > 256 || hdv % 8 || v_row < hdv || v_row % 8) return CBIS_ERR_BAD_SIZE;
-  if (hd <= 0 || hd > 256 || hd % 8 || ps <= 0 || n_head <= 0 || n_kv_head <= 0 || n_head % n_kv_head || nsplit < 1 || nsplit > 32)
+  if (hd <= 0 || hd > 256 || hd % 8 || ps <= 0 || n_head <= 0 || n_kv_head <= 0 || (n_head / v_heads) % n_kv_head || nsplit < 1 || nsplit > 32)
     return CBIS_ERR_BAD_SIZE;
   if (ld % 8 || out_ld % 8 || (k_off >= 0 && (k_off % 8 || v_off % 8)) || ((uintptr_t)qkv & 15) || ((uintptr_t)kc & 15) ||
       ((uintptr_t)vc & 15))
@@ -338,7 +345,7 @@ CBIS_EXPORT int cbis_paged_decode_bf16(const void* qkv, int ld, int k_off, int v
   e = launch_pdl(paged_decode_bf16_kernel<LPK>, grid, dim3(DEC_WARPS * 32), 0, st, (const __nv_bfloat16*)qkv, ld, \
                  k_off, v_off, (__nv_bfloat16*)kc, (__nv_bfloat16*)vc, block_table, max_blocks, row_seq, positions, \
                  slot_mapping, (__nv_bfloat16*)out, out_ld, part, counters, n_head, n_kv_head, hd, ps, scale, window, \
-                 nsplit, hdv, v_row, slopes, sinks, temp_coef, temp_every)
+                 nsplit, hdv, v_row, slopes, sinks, temp_coef, temp_every, rates, v_heads)
   if (chunks <= 2) CBIS_DEC(2);
   else if (chunks <= 4) CBIS_DEC(4);
   else if (chunks <= 8) CBIS_DEC(8);

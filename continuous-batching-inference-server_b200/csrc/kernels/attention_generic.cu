@@ -8,9 +8,11 @@
 // reference keeps [page][page_size][head][head_dim] (kernels/attention.cu:14,80).
 // Keys and values may have different widths (hd, hd_v), the values may be the first hd_v entries of the keys'
 // rows (one cached array for both: vc == kc, v_row == hd), and three things may change the scores and the softmax:
-//   * a distance bias: slope[h] * (p - j) is taken off the scaled score of the key at j for the query at p;
+//   * a distance bias: slope[h] * (p - j), or slope[h] * ln(1 + rate[h] * (p - j)), is taken off the scaled score of the
+//     key at j for the query at p;
 //   * a query temperature: the score of the query at p is also multiplied by 1 + coef * ln(floor((p + 1) / every) + 1);
 //   * a sink: exp(sink[h]) counts once in the softmax's denominator and has no value.
+// With v_heads > 1 every query head attends to the values of every key/value head (head_place in common.cuh).
 #include "attention_merge.cuh"
 
 namespace cbis {
@@ -80,7 +82,7 @@ __global__ void paged_attention_generic_kernel(
     const int* positions, TT* __restrict__ out, int out_ld, int n_rows, int n_head, int n_kv_head,
     int hd, int ps, float scale, int window, int n_chunks, int chunk_keys, float* partial,
     int hd_v, int v_row, const float* __restrict__ slopes, const float* __restrict__ sinks, float temp_coef,
-    int temp_every) {
+    int temp_every, const float* __restrict__ rates, int v_heads) {
   pdl_trigger();
   pdl_wait();
   const int lane = threadIdx.x & 31;
@@ -88,7 +90,7 @@ __global__ void paged_attention_generic_kernel(
   if (wc >= n_rows * n_head * n_chunks) return;
   const int w = wc / n_chunks, chunk = wc % n_chunks;
   const int row = w / n_head, h = w % n_head;
-  const int hk = h / (n_head / n_kv_head);
+  const HeadPlace hp = head_place(h, n_head, n_kv_head, v_heads);
   const int pos = positions[row];
   const int seq = row_seq[row];
   if (seq < 0) {  // a padding row of a fixed-size batch
@@ -98,6 +100,7 @@ __global__ void paged_attention_generic_kernel(
   }
   if (temp_every > 0) scale *= 1.0f + temp_coef * logf((float)((pos + 1) / temp_every + 1));
   const float slope = slopes ? slopes[h] : 0.f;
+  const float* rate = rates ? rates + h : nullptr;
   const int* bt = block_table + (size_t)seq * max_blocks;
   int kend = pos + 1;
   int kstart = first_seen(pos, window);
@@ -111,7 +114,7 @@ __global__ void paged_attention_generic_kernel(
 #pragma unroll
   for (int i = 0; i < NPER; ++i) {
     const int dim = lane + 32 * i;
-    qv[i] = dim < hd ? to_f32(q[(size_t)row * q_ld + h * hd + dim]) : 0.f;
+    qv[i] = dim < hd ? to_f32(q[(size_t)row * q_ld + hp.query * hd + dim]) : 0.f;
     acc[i] = 0.f;
   }
   float m = -INFINITY, l = 0.f;
@@ -126,9 +129,9 @@ __global__ void paged_attention_generic_kernel(
       vptr[u] = nullptr;
       if (j < kend) {
         const int page = bt[j / ps];
-        const size_t token = ((size_t)page * n_kv_head + hk) * ps + (j % ps);
+        const size_t token = ((size_t)page * n_kv_head + hp.key) * ps + (j % ps);
         const TT* kp = kc + token * hd;
-        vptr[u] = vc + token * v_row;
+        vptr[u] = vc + (((size_t)page * n_kv_head + hp.value) * ps + (j % ps)) * v_row;
 #pragma unroll
         for (int i = 0; i < NPER; ++i) {
           const int dim = lane + 32 * i;
@@ -139,7 +142,7 @@ __global__ void paged_attention_generic_kernel(
     }
 #pragma unroll
     for (int u = 0; u < G; ++u)
-      s[u] = (j0 + u < kend) ? fmaf(warp_sum(s[u]), scale, -slope * (float)(pos - (j0 + u))) : -INFINITY;
+      s[u] = (j0 + u < kend) ? fmaf(warp_sum(s[u]), scale, slope != 0.f ? -distance_bias(slope, rate, (float)(pos - (j0 + u))) : 0.f) : -INFINITY;
     float m_new = m;
 #pragma unroll
     for (int u = 0; u < G; ++u) m_new = fmaxf(m_new, s[u]);
@@ -227,7 +230,8 @@ static int launch_generic(const void* q, int q_ld, const void* kc, const void* v
                           int max_blocks, const int* row_seq, const int* positions, void* out, int out_ld,
                           int n_rows, int n_head, int n_kv_head, int hd, int ps, float scale, int window,
                           int n_chunks, int chunk_keys, float* partial, int hd_v, int v_row, const float* slopes,
-                          const float* sinks, float temp_coef, int temp_every, cudaStream_t st) {
+                          const float* sinks, float temp_coef, int temp_every, const float* rates, int v_heads,
+                          cudaStream_t st) {
   const int warps = 4;
   const long long total = (long long)n_rows * n_head * n_chunks;
   const int blocks = (int)((total + warps - 1) / warps);
@@ -236,7 +240,7 @@ static int launch_generic(const void* q, int q_ld, const void* kc, const void* v
   e = launch_pdl(paged_attention_generic_kernel<TT, NPER, (NPER <= 2 ? 16 : (NPER <= 4 ? 8 : (NPER <= 8 ? 4 : 2)))>, dim3(blocks), dim3(warps * 32), 0, st, (const TT*)q, q_ld, \
                  (const TT*)kc, (const TT*)vc, block_table, max_blocks, row_seq, positions, (TT*)out, out_ld, n_rows, \
                  n_head, n_kv_head, hd, ps, scale, window, n_chunks, chunk_keys, partial, hd_v, v_row, slopes, sinks, \
-                 temp_coef, temp_every)
+                 temp_coef, temp_every, rates, v_heads)
   const int widest = hd > hd_v ? hd : hd_v;
   if (widest <= 32) CBIS_LAUNCH(1);
   else if (widest <= 64) CBIS_LAUNCH(2);
@@ -259,11 +263,12 @@ CBIS_EXPORT int cbis_paged_attention_generic(const void* q, int q_ld, const void
                                              int n_kv_head, int hd, int ps, float scale, int window, int dtype,
                                              int n_chunks, int chunk_keys, float* partial, void* stream,
                                              int hd_v, int v_row, const float* slopes, const float* sinks,
-                                             float temp_coef, int temp_every) {
+                                             float temp_coef, int temp_every, const float* rates, int v_heads) {
   if (n_rows <= 0) return CBIS_OK;
   if (hd_v <= 0) hd_v = hd, v_row = hd;      // values as wide as the keys, in an array of their own
   if (hd_v > 512 || v_row < hd_v) return CBIS_ERR_BAD_SIZE;
-  if (hd <= 0 || hd > 512 || ps <= 0 || n_head <= 0 || n_kv_head <= 0 || n_head % n_kv_head) return CBIS_ERR_BAD_SIZE;
+  if (v_heads != 1 && (v_heads != n_kv_head || n_head % v_heads)) return CBIS_ERR_BAD_SIZE;
+  if (hd <= 0 || hd > 512 || ps <= 0 || n_head <= 0 || n_kv_head <= 0 || (n_head / v_heads) % n_kv_head) return CBIS_ERR_BAD_SIZE;
   if (n_chunks < 1 || (n_chunks > 1 && (chunk_keys <= 0 || !partial || hd_v % 4 || out_ld % 4 || ((uintptr_t)partial & 15) ||
                                         ((uintptr_t)out & 15))))
     return CBIS_ERR_BAD_SIZE;
@@ -271,10 +276,10 @@ CBIS_EXPORT int cbis_paged_attention_generic(const void* q, int q_ld, const void
   if (dtype == CBIS_F32)
     return launch_generic<float>(q, q_ld, kc, vc, block_table, max_blocks, row_seq, positions, out, out_ld, n_rows,
                                  n_head, n_kv_head, hd, ps, scale, window, n_chunks, chunk_keys, partial, hd_v, v_row,
-                                 slopes, sinks, temp_coef, temp_every, st);
+                                 slopes, sinks, temp_coef, temp_every, rates, v_heads, st);
   if (dtype == CBIS_BF16)
     return launch_generic<__nv_bfloat16>(q, q_ld, kc, vc, block_table, max_blocks, row_seq, positions, out, out_ld,
                                          n_rows, n_head, n_kv_head, hd, ps, scale, window, n_chunks, chunk_keys, partial, hd_v, v_row,
-                                 slopes, sinks, temp_coef, temp_every, st);
+                                 slopes, sinks, temp_coef, temp_every, rates, v_heads, st);
   return CBIS_ERR_BAD_DTYPE;
 }

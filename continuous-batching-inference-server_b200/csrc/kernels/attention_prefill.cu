@@ -13,7 +13,9 @@
 // Keys and values may be narrower than the tile (hdk, hdv <= HD, multiples of 8: the tiles' columns beyond them are
 // zero), the values may be the first hdv entries of the keys' rows (v_row: elements between two tokens' values),
 // and the scores may carry a distance bias (slope[h] * (p - j) taken off), a query temperature by position and a
-// sink in the denominator, as in the general kernel.
+// sink in the denominator, as in the general kernel.  A bias that grows with the logarithm of the distance (rates) is
+// taken from a table of the tile's 127 distances, made once per key tile; with v_heads > 1 every query head attends to the
+// values of every key/value head (head_place in common.cuh).
 #include "attention_merge.cuh"
 #include <math.h>
 
@@ -67,12 +69,14 @@ paged_prefill_bf16_kernel(const __nv_bfloat16* q, int q_ld, const __nv_bfloat16*
                           __nv_bfloat16* out, int out_ld, int seg0, int n_head, int n_kv_head, int ps_shift,
                           float scale_log2e, int window, int n_chunks, int chunk_keys, float* partial, int row0,
                           int hdk, int hdv, int v_row, const float* __restrict__ slopes,
-                          const float* __restrict__ sinks, float temp_coef, int temp_every) {
+                          const float* __restrict__ sinks, float temp_coef, int temp_every,
+                          const float* __restrict__ rates, int v_heads) {
   constexpr int PITCH = HD + 8;  // elements per shared-memory row: 16 bytes of padding keep ldmatrix conflict-free
   constexpr int KS = HD / 16;    // k-steps of Q*K^T
   constexpr int DT = HD / 8;     // 8-wide column tiles of the output
   constexpr int CHUNKS = HD / 8; // 16-byte pieces per key row
   extern __shared__ __align__(16) unsigned char smem_raw[];
+  __shared__ float s_bias[PF_BM + PF_BN];     // per distance of the tile's first row and key, plus PF_BN - 1: what the bias takes off
   __nv_bfloat16* sK = reinterpret_cast<__nv_bfloat16*>(smem_raw);            // [2][PF_BN][PITCH]
   __nv_bfloat16* sV = sK + 2 * PF_BN * PITCH;                                // [2][PF_BN][PITCH]
   pdl_trigger();
@@ -82,8 +86,9 @@ paged_prefill_bf16_kernel(const __nv_bfloat16* q, int q_ld, const __nv_bfloat16*
   const int chunk = blockIdx.x % n_chunks, tile = gridDim.x / n_chunks - 1 - blockIdx.x / n_chunks;
   const int r_begin = cu_rows[seg], n_rows = cu_rows[seg + 1] - r_begin;
   if (tile * PF_BM >= n_rows) return;
-  const int hk = h / (n_head / n_kv_head);
+  const HeadPlace hp = head_place(h, n_head, n_kv_head, v_heads);
   const int ps = 1 << ps_shift;
+  vc += (ptrdiff_t)(hp.value - hp.key) * ps * v_row;      // a token's row of the value head, counted from its row of the key head
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   const int g = lane >> 2, t = lane & 3;
   const int pos0 = seg_start[seg] + tile * PF_BM;           // position of the tile's first row
@@ -103,8 +108,8 @@ paged_prefill_bf16_kernel(const __nv_bfloat16* q, int q_ld, const __nv_bfloat16*
   const int lo0 = first_seen(p0, window), lo1 = first_seen(p1, window);      // the first key each of the two rows sees
   uint32_t qf[KS][4];
   {
-    const __nv_bfloat16* q0 = q + (size_t)(r_begin + tile * PF_BM + lr0) * q_ld + h * hdk;
-    const __nv_bfloat16* q1 = q + (size_t)(r_begin + tile * PF_BM + lr1) * q_ld + h * hdk;
+    const __nv_bfloat16* q0 = q + (size_t)(r_begin + tile * PF_BM + lr0) * q_ld + hp.query * hdk;
+    const __nv_bfloat16* q1 = q + (size_t)(r_begin + tile * PF_BM + lr1) * q_ld + hp.query * hdk;
     const bool v0 = lr0 < rows_here, v1 = lr1 < rows_here;
 #pragma unroll
     for (int ks = 0; ks < KS; ++ks) {
@@ -139,7 +144,7 @@ paged_prefill_bf16_kernel(const __nv_bfloat16* q, int q_ld, const __nv_bfloat16*
       size_t token = 0;
       if (valid) {
         const int page = bt[j >> ps_shift];
-        token = ((size_t)page * n_kv_head + hk) * ps + (j & (ps - 1));
+        token = ((size_t)page * n_kv_head + hp.key) * ps + (j & (ps - 1));
       }
       const bool in_k = valid && c * 8 < hdk, in_v = valid && c * 8 < hdv;
       cp_async16(dk + r * PITCH + c * 8, kc + (in_k ? token * hdk + c * 8 : 0), in_k);
@@ -156,6 +161,10 @@ paged_prefill_bf16_kernel(const __nv_bfloat16* q, int q_ld, const __nv_bfloat16*
       cp_async_wait<1>();
     } else {
       cp_async_wait<0>();
+    }
+    if (rates) {      // 128 threads, the 127 distances between the tile's rows and keys
+      const int d = pos0 - kt * PF_BN + (int)threadIdx.x - (PF_BN - 1);
+      s_bias[threadIdx.x] = distance_bias(slope2, rates + h, (float)max(d, 0));
     }
     __syncthreads();
     const __nv_bfloat16* tk = sK + (size_t)stage * PF_BN * PITCH;
@@ -188,7 +197,11 @@ paged_prefill_bf16_kernel(const __nv_bfloat16* q, int q_ld, const __nv_bfloat16*
       for (int e = 0; e < 2; ++e) {
         const int j = j0 + nt * 8 + 2 * t + e;
         float a = s[nt][e] * sc0, b2 = s[nt][2 + e] * sc1;
-        if (slopes) {
+        if (rates) {
+          const int at = PF_BN - 1 - (j - j0);
+          a -= s_bias[at + lr0];
+          b2 -= s_bias[at + lr1];
+        } else if (slopes) {
           a = fmaf(-slope2, (float)(p0 - j), a);
           b2 = fmaf(-slope2, (float)(p1 - j), b2);
         }
@@ -291,7 +304,8 @@ CBIS_EXPORT int cbis_paged_prefill_bf16(const void* q, int q_ld, const void* kc,
                                         int max_seg_rows, int n_head, int n_kv_head, int hd, int ps, float scale,
                                         int window, int n_chunks, int chunk_keys, float* partial, const int* positions,
                                         int row0, int n_rows, void* stream, int hd_v, int v_row,
-                                        const float* slopes, const float* sinks, float temp_coef, int temp_every) {
+                                        const float* slopes, const float* sinks, float temp_coef, int temp_every,
+                                        const float* rates, int v_heads) {
   if (n_seg <= 0 || max_seg_rows <= 0) return CBIS_OK;
   // hd: the keys' width; hd_v (0: the keys'): the values'; both multiples of 8, the wider of them rounded up to a
   // multiple of 16 picks the tile
@@ -302,7 +316,8 @@ CBIS_EXPORT int cbis_paged_prefill_bf16(const void* q, int q_ld, const void* kc,
   if (n_chunks < 1 || (n_chunks > 1 && (chunk_keys <= 0 || chunk_keys % PF_BN || !partial || !positions || n_rows <= 0 ||
                                         ((uintptr_t)partial & 15) || out_ld % 4 || ((uintptr_t)out & 7))))
     return CBIS_ERR_BAD_SIZE;
-  if (hd < 16 || hd > 128 || hd % 16 || ps <= 0 || (ps & (ps - 1)) || n_head <= 0 || n_kv_head <= 0 || n_head % n_kv_head)
+  if (hd < 16 || hd > 128 || hd % 16 || ps <= 0 || (ps & (ps - 1)) || n_head <= 0 || n_kv_head <= 0 ||
+      (v_heads != 1 && (v_heads != n_kv_head || n_head % v_heads)) || (n_head / v_heads) % n_kv_head || (rates && !slopes))
     return CBIS_ERR_BAD_SIZE;
   if (q_ld % 8 || out_ld % 2 || ((uintptr_t)q & 15) || ((uintptr_t)kc & 15) || ((uintptr_t)vc & 15) || ((uintptr_t)out & 3))
     return CBIS_ERR_ALIGNMENT;
@@ -324,7 +339,7 @@ CBIS_EXPORT int cbis_paged_prefill_bf16(const void* q, int q_ld, const void* kc,
     e = launch_pdl(kern, grid, dim3(PF_WARPS * 32), smem, st, (const __nv_bfloat16*)q, q_ld, (const __nv_bfloat16*)kc, \
                    (const __nv_bfloat16*)vc, block_table, max_blocks, cu_rows, seg_start, (__nv_bfloat16*)out, out_ld, seg0, \
                    n_head, n_kv_head, ps_shift, scale_log2e, window, n_chunks, chunk_keys, partial, row0, hdk, hd_v,  \
-                   v_row, slopes, sinks, temp_coef, temp_every);                                                      \
+                   v_row, slopes, sinks, temp_coef, temp_every, rates, v_heads);                                                      \
   }
   CBIS_PF(16) CBIS_PF(32) CBIS_PF(48) CBIS_PF(64) CBIS_PF(80) CBIS_PF(96) CBIS_PF(112) CBIS_PF(128)
 #undef CBIS_PF

@@ -150,4 +150,36 @@ __device__ __forceinline__ float activate(float v, int act) {
   return v;
 }
 
+// The inside of a gated feed-forward from the gate's and the up projection's sums.  limit > 0 cuts the gate off at
+// limit from above and the up value at -limit and limit; beta is silu's inner factor, g * sigmoid(beta g); shift is
+// added to the up value.  limit 0, beta 1, shift 0: act(g) * u.
+__device__ __forceinline__ float gated_product(float g, float u, int act, float limit, float beta, float shift) {
+  if (limit > 0.f) {
+    g = fminf(g, limit);
+    u = fminf(fmaxf(u, -limit), limit);
+  }
+  const float a = act == CBIS_ACT_SILU ? g * sigmoid_f32(beta * g) : activate(g, act);
+  return a * (u + shift);
+}
+
+// What a head's distance bias takes off the score of a key `distance` positions back: slope * distance, or, for a head
+// with a rate, slope * ln(1 + rate * distance).
+__device__ __forceinline__ float distance_bias(float slope, const float* rate, float distance) {
+  return rate ? slope * log1pf(*rate * distance) : slope * distance;
+}
+
+// A query head of a launch reads one key head and one value head.  v_heads == 1: both are its own, h / (n_head /
+// n_kv_head).  v_heads == n_kv_head: the launch's head h stands for query head h / v_heads over the values of key/value
+// head h % v_heads, so that every query head meets the values of every key/value head (n_head counts the pairs).
+struct HeadPlace {
+  int query, key, value;
+};
+__device__ __forceinline__ HeadPlace head_place(int h, int n_head, int n_kv_head, int v_heads) {
+  HeadPlace p;
+  p.query = h / v_heads;
+  p.key = p.query / (n_head / v_heads / n_kv_head);
+  p.value = v_heads > 1 ? h % v_heads : p.key;
+  return p;
+}
+
 }  // namespace cbis

@@ -46,11 +46,12 @@ __global__ void rms_norm_kernel(const TI* x, int x_ld, const TG* gate, int gate_
   }
 }
 
-// out[r, c] = act(a[r, c]) * b[r, c]; with `b_rows` b's row is b_rows[r] instead (rows of a table looked up by token;
+// out[r, c] = act(a[r, c]) * b[r, c] (with limit, beta and shift as in gated_product of common.cuh; times row_gate[r], a
+// 32-bit number per row, if there is one); with `b_rows` b's row is b_rows[r] instead (rows of a table looked up by token;
 // an index outside 0 .. b_n_rows - 1 reads as zeros)
 template <typename TT>
 __global__ void gate_mul_kernel(const TT* a, int a_ld, const TT* b, int b_ld, TT* out, int out_ld, int act, int rows,
-                                int n, const int* b_rows, int b_n_rows) {
+                                int n, const int* b_rows, int b_n_rows, float limit, float beta, float shift, const float* row_gate) {
   pdl_trigger();
   pdl_wait();
   const size_t total = (size_t)rows * n;
@@ -65,7 +66,8 @@ __global__ void gate_mul_kernel(const TT* a, int a_ld, const TT* b, int b_ld, TT
       br = there ? (size_t)t : 0;
     }
     const float bv = there ? to_f32(b[br * b_ld + c]) : 0.f;
-    from_f32(out[r * out_ld + c], activate(to_f32(a[r * a_ld + c]), act) * bv);
+    const float v = gated_product(to_f32(a[r * a_ld + c]), bv, act, limit, beta, shift);
+    from_f32(out[r * out_ld + c], row_gate ? v * row_gate[r] : v);
   }
 }
 
@@ -101,7 +103,8 @@ CBIS_EXPORT int cbis_rms_norm(const void* x, int x_ld, int x_dtype, const void* 
 }
 
 CBIS_EXPORT int cbis_gate_mul(const void* a, int a_ld, const void* b, int b_ld, void* out, int out_ld, int act, int rows,
-                              int n, int dtype, void* stream, const int* b_rows, int b_n_rows) {
+                              int n, int dtype, void* stream, const int* b_rows, int b_n_rows, float limit, float beta,
+                              float shift, const float* row_gate) {
   if (rows <= 0 || n <= 0) return CBIS_OK;
   const size_t total = (size_t)rows * n;
   size_t blocks = (total + 255) / 256;
@@ -109,9 +112,11 @@ CBIS_EXPORT int cbis_gate_mul(const void* a, int a_ld, const void* b, int b_ld, 
   cudaStream_t st = (cudaStream_t)stream;
   if (dtype == CBIS_F32)
     return (int)launch_pdl(gate_mul_kernel<float>, dim3((int)blocks), dim3(256), 0, st, (const float*)a, a_ld,
-                           (const float*)b, b_ld, (float*)out, out_ld, act, rows, n, b_rows, b_n_rows);
+                           (const float*)b, b_ld, (float*)out, out_ld, act, rows, n, b_rows, b_n_rows, limit, beta,
+                           shift, row_gate);
   if (dtype == CBIS_BF16)
     return (int)launch_pdl(gate_mul_kernel<__nv_bfloat16>, dim3((int)blocks), dim3(256), 0, st, (const __nv_bfloat16*)a,
-                           a_ld, (const __nv_bfloat16*)b, b_ld, (__nv_bfloat16*)out, out_ld, act, rows, n, b_rows, b_n_rows);
+                           a_ld, (const __nv_bfloat16*)b, b_ld, (__nv_bfloat16*)out, out_ld, act, rows, n, b_rows, b_n_rows, limit, beta,
+                           shift, row_gate);
   return CBIS_ERR_BAD_DTYPE;
 }

@@ -5,7 +5,9 @@
 //     d = delta[s,:] (+ delta_bias)                                           what the part before left
 //     if post_w: d = d / sqrt(mean(d^2) + post_eps) * (post_offset + post_w)   a norm AFTER the part
 //     d = d * delta_scale                                                      a constant on everything that is added
-//     v = x[s,:] + d;  x[s,:] = v                                             the stream moves on (32-bit)
+//     v = x_scale * x[s,:] + d
+//     if stream_w: v = v / sqrt(mean(v^2) + stream_eps) * (stream_offset + stream_w)   a norm of the SUM (post-norm layers)
+//     x[s,:] = v                                                              the stream moves on (32-bit)
 //     out[r,:] = v / sqrt(mean(v^2) + eps) * (offset + w)                      the norm BEFORE the next part
 //   offset 1 is for weights stored around zero, offset 0 for weights stored as they are applied.  With `rows` only
 //   those rows are produced and x is left as it is (the rows whose logits are wanted, before the head).
@@ -19,7 +21,8 @@ template <typename TD, typename TO>
 __global__ void add_rmsnorm_kernel(float* x, const TD* delta, int delta_ld, const float* __restrict__ delta_bias,
                                    const float* __restrict__ post_w, float post_eps, float post_offset,
                                    const float* __restrict__ w, float eps, float offset, TO* out, const int* rows,
-                                   int d, float delta_scale) {
+                                   int d, float delta_scale, float x_scale, const float* __restrict__ stream_w,
+                                   float stream_eps, float stream_offset) {
   extern __shared__ float smem[];
   float* row = smem;           // d floats
   float* dl = smem + d;        // d floats
@@ -44,13 +47,22 @@ __global__ void add_rmsnorm_kernel(float* x, const TD* delta, int delta_ld, cons
   }
   float ss = 0.f;
   for (int c = threadIdx.x; c < d; c += blockDim.x) {
-    float v = xrow[c];
+    float v = __fmul_rn(xrow[c], x_scale);      // on its own: with x_scale 1 the sum rounds as it does without the factor
     if (drow) v += post_w ? dl[c] * dscale * (post_offset + post_w[c]) : dl[c] * dscale;
     row[c] = v;
     ss += v * v;
   }
+  if (stream_w) {
+    const float sinv = 1.0f / sqrtf(block_sum(ss, red) / (float)d + stream_eps);
+    ss = 0.f;
+    for (int c = threadIdx.x; c < d; c += blockDim.x) {
+      const float v = row[c] * sinv * (stream_offset + stream_w[c]);
+      row[c] = v;
+      ss += v * v;
+    }
+  }
   const float inv = w ? 1.0f / sqrtf(block_sum(ss, red) / (float)d + eps) : 1.f;      // no weight: the rows go on as they are
-  const bool write_x = rows == nullptr && drow != nullptr;
+  const bool write_x = rows == nullptr && (drow != nullptr || stream_w != nullptr || x_scale != 1.f);
   TO* orow = out ? out + (size_t)r * d : nullptr;
   for (int c = threadIdx.x; c < d; c += blockDim.x) {
     const float v = row[c];
@@ -86,7 +98,8 @@ template <typename TD, typename TO, int NV>
 __global__ void __launch_bounds__(128)
 add_rmsnorm_reg_kernel(float* x, const TD* delta, int delta_ld, const float* __restrict__ delta_bias,
                        const float* __restrict__ post_w, float post_eps, float post_offset, const float* __restrict__ w,
-                       float eps, float offset, TO* out, const int* rows, int d, float delta_scale) {
+                       float eps, float offset, TO* out, const int* rows, int d, float delta_scale, float x_scale,
+                       const float* __restrict__ stream_w, float stream_eps, float stream_offset) {
   __shared__ float red[33];
   pdl_trigger();
   const int nvec = d >> 2;
@@ -114,6 +127,8 @@ add_rmsnorm_reg_kernel(float* x, const TD* delta, int delta_ld, const float* __r
     v[i] = dl[i] = make_float4(0.f, 0.f, 0.f, 0.f);
     if (c < nvec) {
       v[i] = *reinterpret_cast<const float4*>(xrow + 4 * c);
+      v[i] = make_float4(__fmul_rn(v[i].x, x_scale), __fmul_rn(v[i].y, x_scale), __fmul_rn(v[i].z, x_scale),
+                         __fmul_rn(v[i].w, x_scale));
       if (drow) {
         const float4 t = ld4<TD>(drow + 4 * c);
         dl[i] = make_float4(t.x + db[i].x, t.y + db[i].y, t.z + db[i].z, t.w + db[i].w);
@@ -141,8 +156,22 @@ add_rmsnorm_reg_kernel(float* x, const TD* delta, int delta_ld, const float* __r
       ss += (v[i].x * v[i].x + v[i].y * v[i].y) + (v[i].z * v[i].z + v[i].w * v[i].w);
     }
   }
+  if (stream_w) {
+    const float sinv = 1.0f / sqrtf(block_sum(ss, red) / (float)d + stream_eps);
+    ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const int c = threadIdx.x + i * 128;
+      if (c < nvec) {
+        const float4 sw = *reinterpret_cast<const float4*>(stream_w + 4 * c);
+        v[i] = make_float4(v[i].x * sinv * (stream_offset + sw.x), v[i].y * sinv * (stream_offset + sw.y),
+                           v[i].z * sinv * (stream_offset + sw.z), v[i].w * sinv * (stream_offset + sw.w));
+        ss += (v[i].x * v[i].x + v[i].y * v[i].y) + (v[i].z * v[i].z + v[i].w * v[i].w);
+      }
+    }
+  }
   const float inv = w ? 1.0f / sqrtf(block_sum(ss, red) / (float)d + eps) : 1.f;      // no weight: the rows go on as they are
-  const bool write_x = rows == nullptr && drow != nullptr;
+  const bool write_x = rows == nullptr && (drow != nullptr || stream_w != nullptr || x_scale != 1.f);
 #pragma unroll
   for (int i = 0; i < NV; ++i) {
     const int c = threadIdx.x + i * 128;
@@ -168,7 +197,8 @@ CBIS_EXPORT int cbis_rms_residual_max_width() { return (200 * 1024 / 4 - 64) / 2
 CBIS_EXPORT int cbis_add_rmsnorm(float* x, const void* delta, int delta_ld, int delta_dtype, const float* delta_bias,
                                  const float* post_w, float post_eps, float post_offset, const float* w, float eps,
                                  float offset, void* out, int out_dtype, const int* rows, int n, int d, void* stream,
-                                 float delta_scale) {
+                                 float delta_scale, float x_scale, const float* stream_w, float stream_eps,
+                                 float stream_offset) {
   if (n <= 0) return CBIS_OK;
   if (d <= 0 || d > cbis_rms_residual_max_width()) return CBIS_ERR_BAD_SIZE;
   const int threads = d >= 2048 ? 512 : (d >= 512 ? 256 : 128);
@@ -179,17 +209,19 @@ CBIS_EXPORT int cbis_add_rmsnorm(float* x, const void* delta, int delta_ld, int 
     if (smem > 48 * 1024)                                                                                             \
       cudaFuncSetAttribute(add_rmsnorm_kernel<TD, TO>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);       \
     return (int)launch_pdl(add_rmsnorm_kernel<TD, TO>, dim3(n), dim3(threads), smem, st, x, (const TD*)delta, delta_ld, \
-                           delta_bias, post_w, post_eps, post_offset, w, eps, offset, (TO*)out, rows, d, delta_scale); \
+                           delta_bias, post_w, post_eps, post_offset, w, eps, offset, (TO*)out, rows, d, delta_scale, \
+                           x_scale, stream_w, stream_eps, stream_offset);                                             \
   } while (0)
   const int dd = delta ? delta_dtype : CBIS_F32;
   // rows in registers where every piece is 16 bytes wide and aligned
   const int esz_d = dd == CBIS_F32 ? 4 : 2, esz_o = out_dtype == CBIS_F32 ? 4 : 2;
-  const bool reg = d % 4 == 0 && d <= 128 * 4 * 8 && !((uintptr_t)x & 15) && !((uintptr_t)w & 15) && !((uintptr_t)post_w & 15) &&
+  const bool reg = d % 4 == 0 && d <= 128 * 4 * 8 && !((uintptr_t)x & 15) && !((uintptr_t)w & 15) && !((uintptr_t)post_w & 15) && !((uintptr_t)stream_w & 15) &&
                    !((uintptr_t)delta_bias & 15) && (!delta || (!((uintptr_t)delta & (4 * esz_d - 1)) && delta_ld % 4 == 0)) &&
                    (!out || !((uintptr_t)out & (4 * esz_o - 1)));
 #define CBIS_ARN_REG(TD, TO, NV)                                                                                       \
   return (int)launch_pdl(add_rmsnorm_reg_kernel<TD, TO, NV>, dim3(n), dim3(128), 0, st, x, (const TD*)delta, delta_ld, \
-                         delta_bias, post_w, post_eps, post_offset, w, eps, offset, (TO*)out, rows, d, delta_scale)
+                         delta_bias, post_w, post_eps, post_offset, w, eps, offset, (TO*)out, rows, d, delta_scale, \
+                         x_scale, stream_w, stream_eps, stream_offset)
 #define CBIS_ARN_PICK(TD, TO)                 \
   do {                                        \
     if (d <= 512) CBIS_ARN_REG(TD, TO, 1);    \

@@ -1,29 +1,37 @@
 // A routed mixture of gated feed-forwards.
 //   * route_topk: router logits in 32-bit, a score per expert (sigmoid or softmax), the `top` largest chosen
-//     (ties: the lower index), their weights the scores as they are or divided by their sum;
+//     (ties: the lower index), their weights the scores as they are or divided by their sum; a correction per expert may
+//     join the scores for the choice alone; one more row of the router may give a number per row whose sigmoid is
+//     handed on (the gate of an expert that every row uses);
 //   * routed_gate_up / routed_down: the chosen experts of every row, one (row, choice) pair at a time, the experts'
 //     matrices streamed by warps (a row's result depends on nothing but the row: no other row of the batch and no
 //     position inside it changes a sum's order).  The weight of a choice multiplies the expert's input
 //     (`weight_on_input`), which for the two first products is the same as multiplying their 32-bit sums, or its output.
+//     The gated product inside an expert takes limit, beta and shift (gated_product in common.cuh).
+//   * A chosen index of E or above is an identity expert: its output is the input row itself, times the weight.  It has
+//     no matrices; the kernels that sum a row's choices read the row.
 #include "common.cuh"
 
 namespace cbis {
 
 constexpr int kScoreSigmoid = 0, kScoreSoftmax = 1;
 
-// grid (rows), 256 threads; shared: E floats.  ids [rows, top] int32, weights [rows, top] float.
+// grid (rows), 256 threads; shared: 2 (E + 1) floats.  ids [rows, top] int32, weights [rows, top] float.  correction (may
+// be null): [E], added to the scores for the choice.  side (may be null): [rows], the sigmoid of router row E's logit.
 template <typename TT>
 __global__ void __launch_bounds__(256)
 route_topk_kernel(const TT* h, int h_ld, const TT* __restrict__ router, int* ids, float* weights, int W, int E, int top,
-                  int score, int renormalize, float renorm_eps, float weight_scale) {
+                  int score, int renormalize, float renorm_eps, float weight_scale, const float* __restrict__ correction,
+              float* side) {
   extern __shared__ float z[];
+  float* own = z + E + 1;      // with a correction: the scores, while z holds what the choice is made by
   pdl_trigger();
   pdl_wait();
   const int r = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   const TT* hr = h + (size_t)r * h_ld;
   constexpr int V = 16 / (int)sizeof(TT);      // elements of a 16-byte load
   const bool vec = W % V == 0 && !(((uintptr_t)hr | (uintptr_t)router) & 15);
-  for (int e = warp; e < E; e += 8) {
+  for (int e = warp; e < E + (side ? 1 : 0); e += 8) {
     const TT* wr = router + (size_t)e * W;
     float acc = 0.f;
     if (vec) {
@@ -47,6 +55,7 @@ route_topk_kernel(const TT* h, int h_ld, const TT* __restrict__ router, int* ids
   }
   __syncthreads();
   if (warp != 0) return;
+  if (side && lane == 0) side[r] = sigmoid_f32(z[E]);
   float zmax = -INFINITY, denom = 1.f;
   if (score == kScoreSoftmax) {
     for (int e = lane; e < E; e += 32) zmax = fmaxf(zmax, z[e]);
@@ -54,6 +63,14 @@ route_topk_kernel(const TT* h, int h_ld, const TT* __restrict__ router, int* ids
     float d = 0.f;
     for (int e = lane; e < E; e += 32) d += expf(z[e] - zmax);
     denom = warp_sum(d);
+  }
+  if (correction) {
+    for (int e = lane; e < E; e += 32) {
+      const float sc = score == kScoreSoftmax ? expf(z[e] - zmax) / denom : sigmoid_f32(z[e]);
+      own[e] = sc;
+      z[e] = sc + correction[e];
+    }
+    __syncwarp();
   }
   float total = 0.f;
   for (int k = 0; k < top; ++k) {
@@ -71,7 +88,7 @@ route_topk_kernel(const TT* h, int h_ld, const TT* __restrict__ router, int* ids
       if (ob > best || (ob == best && oa < arg)) { best = ob; arg = oa; }
     }
     if (arg >= E) arg = k < E ? k : 0;          // rows of not-a-numbers (padding): any valid expert
-    const float sc = score == kScoreSoftmax ? expf(best - zmax) / denom : sigmoid_f32(best);
+    const float sc = correction ? own[arg] : (score == kScoreSoftmax ? expf(best - zmax) / denom : sigmoid_f32(best));
     total += sc;
     if (lane == 0) {
       ids[(size_t)r * top + k] = arg;
@@ -92,17 +109,19 @@ route_topk_kernel(const TT* h, int h_ld, const TT* __restrict__ router, int* ids
 template <typename TT>
 __global__ void __launch_bounds__(256)
 routed_gate_up_kernel(const TT* h, int h_ld, const TT* __restrict__ gate_up, const int* ids, const float* weights,
-                      TT* hid, int W, int F, int top, int act, int weight_on_input) {
+                      TT* hid, int W, int F, int top, int act, int weight_on_input, int E, float limit, float beta,
+                      float shift) {
   extern __shared__ float hs[];
   pdl_trigger();
   pdl_wait();
   const int pair = blockIdx.x, row = pair / top;
+  const int e = ids[pair];
+  if (e >= E) return;         // an identity expert: nothing to compute
   const TT* hr = h + (size_t)row * h_ld;
   for (int k = threadIdx.x; k < W; k += 256) hs[k] = to_f32(hr[k]);
   __syncthreads();
   const int lane = threadIdx.x & 31, f = blockIdx.y * 8 + (threadIdx.x >> 5);
   if (f >= F) return;
-  const int e = ids[pair];
   const TT* wg = gate_up + ((size_t)e * 2 * F + f) * W;
   const TT* wu = wg + (size_t)F * W;
   float g = 0.f, u = 0.f;
@@ -129,17 +148,17 @@ routed_gate_up_kernel(const TT* h, int h_ld, const TT* __restrict__ gate_up, con
   u = warp_sum(u);
   if (lane == 0) {
     const float s = weight_on_input ? weights[pair] : 1.f;
-    from_f32(hid[(size_t)pair * F + f], activate(s * g, act) * (s * u));
+    from_f32(hid[(size_t)pair * F + f], gated_product(s * g, s * u, act, limit, beta, shift));
   }
 }
 
 // grid (rows, ceil(W / 8)), 256 threads: out[row, n] = sum over the row's choices k of
 //   (weight on output ? weight : 1) * (Wd_e[n, :] . hid[row * top + k, :]),   down: [E, W, F].  out is 32-bit and is
-// overwritten, or added to with `accumulate`.
+// overwritten, or added to with `accumulate`.  A choice of E or above adds weight * h[row, n].
 template <typename TT>
 __global__ void __launch_bounds__(256)
 routed_down_kernel(const TT* hid, const TT* __restrict__ down, const int* ids, const float* weights, float* out,
-                   int out_ld, int W, int F, int top, int weight_on_input, int accumulate) {
+                   int out_ld, int W, int F, int top, int weight_on_input, int accumulate, int E, const TT* h, int h_ld) {
   pdl_trigger();
   pdl_wait();
   const int row = blockIdx.x, lane = threadIdx.x & 31, n = blockIdx.y * 8 + (threadIdx.x >> 5);
@@ -147,6 +166,10 @@ routed_down_kernel(const TT* hid, const TT* __restrict__ down, const int* ids, c
   float total = 0.f;
   for (int k = 0; k < top; ++k) {
     const int pair = row * top + k;
+    if (ids[pair] >= E) {      // uniform over the warp
+      total += weights[pair] * to_f32(h[(size_t)row * h_ld + n]);
+      continue;
+    }
     const TT* wd = down + ((size_t)ids[pair] * W + n) * F;
     const TT* hp = hid + (size_t)pair * F;
     float acc = 0.f;
@@ -163,7 +186,7 @@ routed_down_kernel(const TT* hid, const TT* __restrict__ down, const int* ids, c
       for (int f = lane; f < F; f += 32) acc = fmaf(to_f32(wd[f]), to_f32(hp[f]), acc);
     }
     acc = warp_sum(acc);
-    total += weight_on_input ? acc : acc * weights[pair];
+    total = weight_on_input ? total + acc : fmaf(acc, weights[pair], total);
   }
   if (lane == 0) {
     float* o = out + (size_t)row * out_ld + n;
@@ -236,7 +259,8 @@ template <bool DUAL>
 __global__ void __launch_bounds__(256)
 routed_tiles_kernel(const __nv_bfloat16* A, int a_ld, const __nv_bfloat16* __restrict__ Bw, const int* sorted,
                     const float* weights, const int* tile_expert, const int* tile_start, const int* tile_rows,
-                    const int* n_tiles, void* out, int out_ld, int N, int K, int top, int act, int weight_on_input) {
+                    const int* n_tiles, void* out, int out_ld, int N, int K, int top, int act, int weight_on_input,
+                    float limit, float beta, float shift) {
   __shared__ __align__(16) __nv_bfloat16 As[kTileM][kLd];
   __shared__ __align__(16) __nv_bfloat16 Bs[DUAL ? 2 : 1][kTileN][kLd];
   __shared__ int pair_of[kTileM];
@@ -331,7 +355,7 @@ routed_tiles_kernel(const __nv_bfloat16* A, int a_ld, const __nv_bfloat16* __res
           if (DUAL) {
             const float s = weight_on_input ? w : 1.f;
             from_f32(static_cast<__nv_bfloat16*>(out)[(size_t)pair * out_ld + n],
-                     activate(s * v0, act) * (s * acc[DUAL ? 1 : 0][mt][j][half * 2 + i]));
+                     gated_product(s * v0, s * acc[DUAL ? 1 : 0][mt][j][half * 2 + i], act, limit, beta, shift));
           } else {
             static_cast<float*>(out)[(size_t)pair * out_ld + n] = weight_on_input ? v0 : w * v0;
           }
@@ -339,8 +363,10 @@ routed_tiles_kernel(const __nv_bfloat16* A, int a_ld, const __nv_bfloat16* __res
     }
 }
 
-// out[row, n] (+)= y[row * top + 0, n] + y[row * top + 1, n] + ..., in that order; 32-bit.
-__global__ void routed_combine_kernel(const float* y, float* out, int out_ld, int rows, int W, int top, int accumulate) {
+// out[row, n] (+)= y[row * top + 0, n] + y[row * top + 1, n] + ..., in that order; 32-bit.  A choice of E or above has no
+// y: it adds weight * h[row, n].
+__global__ void routed_combine_kernel(const float* y, float* out, int out_ld, int rows, int W, int top, int accumulate,
+                                      const int* ids, const float* weights, int E, const __nv_bfloat16* h, int h_ld) {
   pdl_trigger();
   pdl_wait();
   const size_t total = (size_t)rows * W;
@@ -348,7 +374,8 @@ __global__ void routed_combine_kernel(const float* y, float* out, int out_ld, in
     const size_t r = i / W;
     const int n = (int)(i % W);
     float v = 0.f;
-    for (int k = 0; k < top; ++k) v += y[(r * top + k) * W + n];
+    for (int k = 0; k < top; ++k)
+      v += ids[r * top + k] < E ? y[(r * top + k) * W + n] : weights[r * top + k] * to_f32(h[r * h_ld + n]);
     float* o = out + r * out_ld + n;
     *o = accumulate ? *o + v : v;
   }
@@ -372,7 +399,7 @@ CBIS_EXPORT long long cbis_routed_plan_ints(int pairs, int E) {
 CBIS_EXPORT int cbis_routed_tiles(const void* h, int h_ld, const void* gate_up, const void* down, const int* ids,
                                   const float* weights, int* plan, void* hid, float* y, float* out, int out_ld, int rows,
                                   int W, int F, int E, int top, int act, int weight_on_input, int accumulate,
-                                  void* stream) {
+                                  void* stream, int identity, float limit, float beta, float shift) {
   if (rows <= 0) return CBIS_OK;
   if (W <= 0 || F <= 0 || E <= 0 || top <= 0) return CBIS_ERR_BAD_SIZE;
   if (W % 8 || F % 8 || h_ld % 8) return CBIS_ERR_ALIGNMENT;
@@ -393,42 +420,43 @@ CBIS_EXPORT int cbis_routed_tiles(const void* h, int h_ld, const void* gate_up, 
   typedef const __nv_bfloat16* bp;
   err = launch_pdl(routed_tiles_kernel<true>, dim3(max_tiles, (F + kTileN - 1) / kTileN), dim3(256), 0, st, (bp)h, h_ld,
                    (bp)gate_up, (const int*)sorted, weights, (const int*)tile_expert, (const int*)tile_start,
-                   (const int*)tile_rows, (const int*)n_tiles, hid, F, F, W, top, act, weight_on_input);
+                   (const int*)tile_rows, (const int*)n_tiles, hid, F, F, W, top, act, weight_on_input, limit, beta, shift);
   if (err != cudaSuccess) return (int)err;
-  const bool direct = top == 1 && !accumulate;
+  const bool direct = top == 1 && !accumulate && identity == 0;
   err = launch_pdl(routed_tiles_kernel<false>, dim3(max_tiles, (W + kTileN - 1) / kTileN), dim3(256), 0, st, (bp)hid, F,
                    (bp)down, (const int*)sorted, weights, (const int*)tile_expert, (const int*)tile_start,
                    (const int*)tile_rows, (const int*)n_tiles, (void*)(direct ? out : y), direct ? out_ld : W, W, F, top,
-                   act, weight_on_input);
+                   act, weight_on_input, limit, beta, shift);
   if (err != cudaSuccess || direct) return (int)err;
   const size_t total = (size_t)rows * W;
   size_t blocks = (total + 255) / 256;
   if (blocks > 148 * 16) blocks = 148 * 16;
   return (int)launch_pdl(routed_combine_kernel, dim3((int)blocks), dim3(256), 0, st, (const float*)y, out, out_ld, rows, W,
-                         top, accumulate);
+                         top, accumulate, ids, weights, E, (bp)h, h_ld);
 }
 
 CBIS_EXPORT int cbis_route_topk(const void* h, int h_ld, const void* router, int* ids, float* weights, int rows, int W,
                                 int E, int top, int score, int renormalize, int dtype, void* stream, float renorm_eps,
-                                float weight_scale) {
+                                float weight_scale, const float* correction, float* side) {
   if (rows <= 0) return CBIS_OK;
   if (W <= 0 || E <= 0 || top <= 0 || top > E || (score != kScoreSigmoid && score != kScoreSoftmax)) return CBIS_ERR_BAD_SIZE;
-  if (E > 8192) return CBIS_ERR_TOO_LARGE;
+  if (E > 6000) return CBIS_ERR_TOO_LARGE;
   cudaStream_t st = (cudaStream_t)stream;
-  const size_t smem = (size_t)E * sizeof(float);
+  const size_t smem = (size_t)2 * (E + 1) * sizeof(float);
   if (dtype == CBIS_F32)
     return (int)launch_pdl(route_topk_kernel<float>, dim3(rows), dim3(256), smem, st, (const float*)h, h_ld,
-                           (const float*)router, ids, weights, W, E, top, score, renormalize, renorm_eps, weight_scale);
+                           (const float*)router, ids, weights, W, E, top, score, renormalize, renorm_eps, weight_scale,
+                           correction, side);
   if (dtype == CBIS_BF16)
     return (int)launch_pdl(route_topk_kernel<__nv_bfloat16>, dim3(rows), dim3(256), smem, st, (const __nv_bfloat16*)h, h_ld,
                            (const __nv_bfloat16*)router, ids, weights, W, E, top, score, renormalize, renorm_eps,
-                           weight_scale);
+                           weight_scale, correction, side);
   return CBIS_ERR_BAD_DTYPE;
 }
 
 CBIS_EXPORT int cbis_routed_gate_up(const void* h, int h_ld, const void* gate_up, const int* ids, const float* weights,
                                     void* hid, int rows, int W, int F, int top, int act, int weight_on_input, int dtype,
-                                    void* stream) {
+                                    void* stream, int E, float limit, float beta, float shift) {
   if (rows <= 0) return CBIS_OK;
   if (W <= 0 || F <= 0 || top <= 0) return CBIS_ERR_BAD_SIZE;
   if (W > 12288 || F > 8 * 65535) return CBIS_ERR_TOO_LARGE;
@@ -437,17 +465,18 @@ CBIS_EXPORT int cbis_routed_gate_up(const void* h, int h_ld, const void* gate_up
   const size_t smem = (size_t)W * sizeof(float);
   if (dtype == CBIS_F32)
     return (int)launch_pdl(routed_gate_up_kernel<float>, grid, dim3(256), smem, st, (const float*)h, h_ld,
-                           (const float*)gate_up, ids, weights, (float*)hid, W, F, top, act, weight_on_input);
+                           (const float*)gate_up, ids, weights, (float*)hid, W, F, top, act, weight_on_input, E, limit,
+                           beta, shift);
   if (dtype == CBIS_BF16)
     return (int)launch_pdl(routed_gate_up_kernel<__nv_bfloat16>, grid, dim3(256), smem, st, (const __nv_bfloat16*)h, h_ld,
                            (const __nv_bfloat16*)gate_up, ids, weights, (__nv_bfloat16*)hid, W, F, top, act,
-                           weight_on_input);
+                           weight_on_input, E, limit, beta, shift);
   return CBIS_ERR_BAD_DTYPE;
 }
 
 CBIS_EXPORT int cbis_routed_down(const void* hid, const void* down, const int* ids, const float* weights, float* out,
                                  int out_ld, int rows, int W, int F, int top, int weight_on_input, int accumulate,
-                                 int dtype, void* stream) {
+                                 int dtype, void* stream, int E, const void* h, int h_ld) {
   if (rows <= 0) return CBIS_OK;
   if (W <= 0 || F <= 0 || top <= 0) return CBIS_ERR_BAD_SIZE;
   if (W > 8 * 65535) return CBIS_ERR_TOO_LARGE;
@@ -455,9 +484,10 @@ CBIS_EXPORT int cbis_routed_down(const void* hid, const void* down, const int* i
   const dim3 grid(rows, (W + 7) / 8);
   if (dtype == CBIS_F32)
     return (int)launch_pdl(routed_down_kernel<float>, grid, dim3(256), 0, st, (const float*)hid, (const float*)down, ids,
-                           weights, out, out_ld, W, F, top, weight_on_input, accumulate);
+                           weights, out, out_ld, W, F, top, weight_on_input, accumulate, E, (const float*)h, h_ld);
   if (dtype == CBIS_BF16)
     return (int)launch_pdl(routed_down_kernel<__nv_bfloat16>, grid, dim3(256), 0, st, (const __nv_bfloat16*)hid,
-                           (const __nv_bfloat16*)down, ids, weights, out, out_ld, W, F, top, weight_on_input, accumulate);
+                           (const __nv_bfloat16*)down, ids, weights, out, out_ld, W, F, top, weight_on_input, accumulate, E,
+                           (const __nv_bfloat16*)h, h_ld);
   return CBIS_ERR_BAD_DTYPE;
 }

@@ -510,7 +510,7 @@ def generic_key_chunks(rows: int, n_head: int, max_context: int, head_dim: int):
 
 def paged_attention_generic(q, k_cache, v_cache, block_table, row_seq, positions, out, n_head, n_kv_head,
                             head_dim, page_size, scale, window=0, chunks=(1, 0), partial=None, v_head_dim=0,
-                            slopes=None, sinks=None, q_temp=None):
+                            slopes=None, sinks=None, q_temp=None, rates=None, v_heads=1):
     """Attention of every row over its request's pages: keys max(0,p-window+1)..p for the query at p.
     ``window`` is one signed number in every attention kernel: 0 every key up to p; w > 0 a sliding window of w keys;
     w < 0 the keys of p's own block of -w positions, p - p mod (-w) .. p, blocks counted from position 0.
@@ -520,12 +520,15 @@ def paged_attention_generic(q, k_cache, v_cache, block_table, row_seq, positions
     the value pages may be the key pages themselves, whose rows' first entries are then the values.  ``slopes`` (32-bit,
     per head): slope * (p - j) is taken off the score of the key at j.  ``sinks`` (32-bit, per head): exp(sink) joins
     the softmax's denominator.  ``q_temp`` = (coef, every): the scores of the query at p are multiplied by
-    1 + coef * ln(floor((p + 1) / every) + 1)."""
+    1 + coef * ln(floor((p + 1) / every) + 1).  ``rates`` (32-bit, per head, with ``slopes``): the bias is
+    slope * ln(1 + rate * (p - j)) instead.  ``v_heads`` = n_kv_head: the launch's head h is query head h / v_heads over
+    the values of key/value head h % v_heads (``n_head``, and every array per head, counts these pairs; q holds
+    n_head / v_heads heads)."""
     _need_cuda(q, k_cache, v_cache, block_table, row_seq, positions, out, partial)
     T = q.shape[0]
     if head_dim > ATTENTION_MAX_HEAD_DIM:
         raise KernelError(f"attention: head_dim={head_dim} is above the kernel's limit of {ATTENTION_MAX_HEAD_DIM}")
-    if n_head % n_kv_head:
+    if n_head % (n_kv_head * v_heads):
         raise KernelError(f"attention: n_head={n_head} is not a multiple of n_kv_head={n_kv_head}")
     assert q.stride(1) == 1 and out.stride(1) == 1 and block_table.dtype == torch.int32
     assert block_table.is_contiguous() and row_seq.dtype == torch.int32 and positions.dtype == torch.int32
@@ -534,7 +537,7 @@ def paged_attention_generic(q, k_cache, v_cache, block_table, row_seq, positions
     v_row = v_cache.shape[-1]
     if vd > v_row:
         raise KernelError(f"attention: values of {vd} do not fit pages of rows of {v_row}")
-    for t in (slopes, sinks):
+    for t in (slopes, sinks, rates):
         assert t is None or (t.dtype == torch.float32 and t.numel() == n_head and t.is_cuda)
     if n_chunks > 1:
         assert partial.dtype == torch.float32 and partial.numel() >= T * n_head * n_chunks * (vd + 4)
@@ -546,7 +549,7 @@ def paged_attention_generic(q, k_cache, v_cache, block_table, row_seq, positions
         _ptr(row_seq), _ptr(positions), _ptr(out), c_int(out.stride(0)), c_int(T), c_int(n_head), c_int(n_kv_head),
         c_int(head_dim), c_int(page_size), c_float(scale), c_int(window), c_int(dtype_code(q.dtype)),
         c_int(n_chunks), c_int(chunk_keys), _ptr(partial), _stream(), c_int(vd), c_int(v_row), _ptr(slopes), _ptr(sinks),
-        c_float(coef), c_int(int(every)))
+        c_float(coef), c_int(int(every)), _ptr(rates), c_int(v_heads))
     _check(st, "paged_attention_generic", f"T={T} heads={n_head}/{n_kv_head} head_dim={head_dim} page={page_size} "
                                           f"chunks={n_chunks}x{chunk_keys}")
 
@@ -567,11 +570,11 @@ def decode_scratch_floats(rows: int, n_head: int, head_dim: int, nsplit: int) ->
 
 def paged_decode_bf16(qkv, k_off, v_off, k_cache, v_cache, block_table, row_seq, positions, slot_mapping, out,
                       scratch, counters, n_head, n_kv_head, head_dim, page_size, scale, window, nsplit, v_head_dim=0,
-                      slopes=None, sinks=None, q_temp=None):
+                      slopes=None, sinks=None, q_temp=None, rates=None, v_heads=1):
     """Decode attention (one query per row) with the keys split ``nsplit`` ways; with ``k_off >= 0`` the
     current token's key/value are taken from ``qkv`` and stored into the cache by the same kernel.
     ``scratch``: ``decode_scratch_floats`` floats; ``counters``: rows*n_head int32, zero before the
-    first launch (every launch leaves them zero).  ``v_head_dim``, ``slopes``, ``sinks``, ``q_temp``: as in
+    first launch (every launch leaves them zero).  ``v_head_dim``, ``slopes``, ``sinks``, ``q_temp``, ``rates``, ``v_heads``: as in
     ``paged_attention_generic`` (widths multiples of 8 up to 256; the scratch is then sized by the values' width)."""
     _need_cuda(qkv, k_cache, v_cache, block_table, row_seq, positions, slot_mapping, out, scratch, counters, slopes, sinks)
     rows = qkv.shape[0]
@@ -579,7 +582,7 @@ def paged_decode_bf16(qkv, k_off, v_off, k_cache, v_cache, block_table, row_seq,
     if head_dim % 8 or head_dim > 256 or vd % 8 or vd > 256:
         raise KernelError(f"decode attention: widths {head_dim} and {vd} must be multiples of 8, at most 256")
     assert qkv.dtype == torch.bfloat16 and k_cache.dtype == torch.bfloat16 and out.dtype == torch.bfloat16
-    for t in (slopes, sinks):
+    for t in (slopes, sinks, rates):
         assert t is None or (t.dtype == torch.float32 and t.numel() == n_head)
     coef, every = q_temp if q_temp else (0.0, 0)
     if nsplit > 1:
@@ -590,18 +593,20 @@ def paged_decode_bf16(qkv, k_off, v_off, k_cache, v_cache, block_table, row_seq,
         c_int(block_table.shape[1]), _ptr(row_seq), _ptr(positions), _ptr(slot_mapping), _ptr(out),
         c_int(out.stride(0)), _ptr(scratch), _ptr(counters), c_int(rows), c_int(n_head), c_int(n_kv_head),
         c_int(head_dim), c_int(page_size), c_float(scale), c_int(window), c_int(nsplit), _stream(),
-        c_int(int(v_head_dim)), c_int(v_cache.shape[-1]), _ptr(slopes), _ptr(sinks), c_float(coef), c_int(int(every)))
+        c_int(int(v_head_dim)), c_int(v_cache.shape[-1]), _ptr(slopes), _ptr(sinks), c_float(coef), c_int(int(every)),
+        _ptr(rates), c_int(v_heads))
     _check(st, "paged_decode_bf16", f"rows={rows} heads={n_head}/{n_kv_head} head_dim={head_dim} splits={nsplit}")
 
 
 def paged_prefill_bf16(q, k_cache, v_cache, block_table, cu_rows, seg_start, out, seg0, n_seg, max_seg_rows,
                        n_head, n_kv_head, head_dim, page_size, scale, window=0, chunks=(1, 0), partial=None,
-                       positions=None, row0=0, n_rows=0, v_head_dim=0, slopes=None, sinks=None, q_temp=None):
+                       positions=None, row0=0, n_rows=0, v_head_dim=0, slopes=None, sinks=None, q_temp=None, rates=None,
+                       v_heads=1):
     """Attention of the segments seg0..seg0+n_seg-1 (runs of rows given by ``cu_rows``, first positions
     ``seg_start``) over their pages, on the tensor cores.  Head sizes 16, 32, ... 128, page sizes 2^k.
     With ``v_head_dim`` keys and values may have different widths, multiples of 8 up to 128 (the value pages may be
-    the key pages: a row's first entries are then its values); ``slopes``, ``sinks``, ``q_temp``: as in
-    ``paged_attention_generic``.
+    the key pages: a row's first entries are then its values); ``slopes``, ``sinks``, ``q_temp``, ``rates``, ``v_heads``: as
+    in ``paged_attention_generic``.
     ``chunks`` = (n, keys) from ``prefill_key_chunks`` cuts the keys n ways over more blocks (every context of the
     step below n * keys); ``partial`` then holds ``n_rows * n_head * n * (head_dim + 4)`` floats, ``positions`` the
     position of every row, ``row0`` and ``n_rows`` name the rows of these segments."""
@@ -616,7 +621,7 @@ def paged_prefill_bf16(q, k_cache, v_cache, block_table, cu_rows, seg_start, out
     assert q.dtype == torch.bfloat16 and k_cache.dtype == torch.bfloat16 and out.dtype == torch.bfloat16
     assert q.stride(1) == 1 and out.stride(1) == 1 and block_table.is_contiguous()
     v_row = v_cache.shape[-1]
-    for t in (slopes, sinks):
+    for t in (slopes, sinks, rates):
         assert t is None or (t.dtype == torch.float32 and t.numel() == n_head and t.is_cuda)
     coef, every = q_temp if q_temp else (0.0, 0)
     n_chunks, chunk_keys = chunks
@@ -628,7 +633,8 @@ def paged_prefill_bf16(q, k_cache, v_cache, block_table, cu_rows, seg_start, out
         _ptr(cu_rows), _ptr(seg_start), _ptr(out), c_int(out.stride(0)), c_int(seg0), c_int(n_seg),
         c_int(max_seg_rows), c_int(n_head), c_int(n_kv_head), c_int(head_dim), c_int(page_size), c_float(scale),
         c_int(window), c_int(n_chunks), c_int(chunk_keys), _ptr(partial), _ptr(positions), c_int(row0), c_int(n_rows),
-        _stream(), c_int(vd), c_int(v_row), _ptr(slopes), _ptr(sinks), c_float(coef), c_int(int(every)))
+        _stream(), c_int(vd), c_int(v_row), _ptr(slopes), _ptr(sinks), c_float(coef), c_int(int(every)), _ptr(rates),
+        c_int(v_heads))
     _check(st, "paged_prefill_bf16", f"segments={n_seg} heads={n_head}/{n_kv_head} head_dim={head_dim} page={page_size} "
                                      f"chunks={n_chunks}x{chunk_keys}")
 
@@ -813,18 +819,22 @@ def rms_norm(x, weight, eps, out, parts: int = 1, gate=None, gate_act="silu", ga
     _check(st, "rms_norm", f"rows={rows} width={n} parts={parts}")
 
 
-def gate_mul(a, b, act, out, b_rows=None):
+def gate_mul(a, b, act, out, b_rows=None, limit: float = 0.0, beta: float = 1.0, shift: float = 0.0, row_gate=None):
     """out = act(a) * b element by element (32-bit arithmetic, one rounding); a, b, out: ``[rows, n]`` of one type,
     views with unit column stride are fine.  With ``b_rows`` (int32, one per row) b is a table ``[*, n]`` and row r
-    takes b[b_rows[r]] (a token's row of a table; an index outside the table reads as zeros)."""
+    takes b[b_rows[r]] (a token's row of a table; an index outside the table reads as zeros).  ``limit`` > 0: a is cut off
+    at limit from above and b at -limit and limit first; ``beta``: silu is a * sigmoid(beta a); ``shift`` is added to b;
+    ``row_gate`` (32-bit, one per row) multiplies the row."""
     _need_cuda(a, b, out, b_rows)
     rows, n = a.shape
     assert out.shape == a.shape and a.dtype == b.dtype == out.dtype and b.shape[1] == n
     assert b.shape == a.shape if b_rows is None else (b_rows.dtype == torch.int32 and b_rows.shape[0] >= rows)
     assert a.stride(1) == 1 and b.stride(1) == 1 and out.stride(1) == 1
+    assert row_gate is None or (row_gate.dtype == torch.float32 and row_gate.is_contiguous() and row_gate.numel() >= rows)
     st = kernels().cbis_gate_mul(_ptr(a), c_int(a.stride(0)), _ptr(b), c_int(b.stride(0)), _ptr(out), c_int(out.stride(0)),
                                  c_int(ACT[act]), c_int(rows), c_int(n), c_int(dtype_code(a.dtype)), _stream(),
-                                 _ptr(b_rows), c_int(b.shape[0]))
+                                 _ptr(b_rows), c_int(b.shape[0]), c_float(limit), c_float(beta), c_float(shift),
+                                 _ptr(row_gate))
     _check(st, "gate_mul", f"rows={rows} n={n}")
 
 
@@ -832,12 +842,15 @@ RMS_RESIDUAL_MAX_WIDTH = (200 * 1024 // 4 - 64) // 2     # the widest row add_rm
 MATRIX_MEMORY_MAX_DIM = 512                              # the widest key of the matrix memory (cbis_matrix_memory_max_dim())
 
 
-def add_rmsnorm(x, delta, delta_bias, post, weight, eps, offset, out, rows=None, delta_scale: float = 1.0):
+def add_rmsnorm(x, delta, delta_bias, post, weight, eps, offset, out, rows=None, delta_scale: float = 1.0,
+                x_scale: float = 1.0, stream=None):
     """One pass over the rows of the 32-bit residual stream ``x``: what a part left (``delta``, 32-bit or the compute
     type, plus ``delta_bias`` per column) is, with ``post`` = (weight, eps, offset), first divided by its own root mean
     square and multiplied by (offset + weight); it is added to x in place; and ``out`` takes x / sqrt(mean(x^2) + eps)
     * (offset + weight) (``weight`` None: x itself; ``out`` None: nothing).  With ``rows`` (int32) only those rows
-    are produced and x is not changed.  ``delta_scale`` multiplies what is added (after its own norm, if it has one)."""
+    are produced and x is not changed.  ``delta_scale`` multiplies what is added (after its own norm, if it has one).
+    ``x_scale`` multiplies x before the addition, and with ``stream`` = (weight, eps, offset) the SUM is divided by its root
+    mean square and multiplied by (offset + weight) before it becomes x (layers whose norm stands after the addition)."""
     _need_cuda(x, delta, delta_bias, weight, out, rows)
     d = x.shape[1]
     assert x.dtype == torch.float32 and x.is_contiguous()
@@ -845,13 +858,14 @@ def add_rmsnorm(x, delta, delta_bias, post, weight, eps, offset, out, rows=None,
     assert out is None or (out.is_contiguous() and out.shape == (n, d))
     assert delta is None or (delta.shape == x.shape and delta.stride(1) == 1)
     pw, peps, poff = post if post is not None else (None, 0.0, 0.0)
-    for t in (delta_bias, pw, weight):
+    sw, seps, soff = stream if stream is not None else (None, 0.0, 0.0)
+    for t in (delta_bias, pw, weight, sw):
         assert t is None or (t.dtype == torch.float32 and t.numel() == d and t.is_contiguous())
     st = kernels().cbis_add_rmsnorm(_ptr(x), _ptr(delta), c_int(delta.stride(0) if delta is not None else 0),
                                     c_int(dtype_code(delta.dtype) if delta is not None else 0), _ptr(delta_bias), _ptr(pw),
                                     c_float(peps), c_float(poff), _ptr(weight), c_float(eps), c_float(offset), _ptr(out),
                                     c_int(dtype_code(out.dtype) if out is not None else 0), _ptr(rows), c_int(n), c_int(d),
-                                    _stream(), c_float(delta_scale))
+                                    _stream(), c_float(delta_scale), c_float(x_scale), _ptr(sw), c_float(seps), c_float(soff))
     _check(st, "add_rmsnorm", f"rows={n} width={d}")
 
 
@@ -1033,6 +1047,40 @@ def qk_prepare(buf, q_off, q_heads, k_off, k_heads, width, q_weight, k_weight, e
     _check(st, "qk_prepare", f"rows={rows} heads={q_heads}/{k_heads} width={width} rot_dims={rot_dims}")
 
 
+def qk_head_norm(buf, q_off, q_heads, k_off, k_heads, width, q_weight, k_weight, eps):
+    """Every head of q (``q_heads`` x ``width`` columns of ``buf`` from ``q_off``, in place) divided by its own root mean
+    square and multiplied by ``q_weight`` (``width`` numbers, shared by all heads); the same for k (``k_heads`` 0: none).
+    32-bit arithmetic, one rounding; heads up to 512 wide."""
+    _need_cuda(buf, q_weight, k_weight)
+    assert buf.stride(1) == 1 and q_off + q_heads * width <= buf.shape[1] and k_off + k_heads * width <= buf.shape[1]
+    for w, n in ((q_weight, q_heads), (k_weight, k_heads)):
+        assert n == 0 or (w.dtype == torch.float32 and w.numel() == width and w.is_contiguous())
+    st = kernels().cbis_qk_head_norm(_ptr(buf), c_int(buf.stride(0)), c_int(q_off), c_int(q_heads), c_int(k_off), c_int(k_heads),
+                                     c_int(width), _ptr(q_weight), _ptr(k_weight), c_float(eps), c_int(buf.shape[0]),
+                                     c_int(dtype_code(buf.dtype)), _stream())
+    _check(st, "qk_head_norm", f"rows={buf.shape[0]} heads={q_heads}/{k_heads} width={width}")
+
+
+MIX_HEADS_MAX_HEADS = 224        # the most heads mix_heads takes (cbis_mix_heads_max_heads() says the same)
+
+
+def mix_heads(o, talk, n_head, n_kv_head, v_dim, out, gate=None):
+    """out[:, h] = sum over g of talk[h, g] * o[:, g, kv(h)], kv(h) = h // (n_head / n_kv_head), times sigmoid(gate[:, h])
+    element by element if a gate is given.  ``o`` ``[rows, n_head * n_kv_head * v_dim]``: what query head g's weights make of
+    the values of every key/value head, side by side; talk 32-bit ``[n_head, n_head]``; out and gate
+    ``[rows, n_head * v_dim]`` of o's type.  Sums in 32-bit, one rounding."""
+    _need_cuda(o, talk, out, gate)
+    rows = o.shape[0]
+    assert o.shape[1] == n_head * n_kv_head * v_dim and o.stride(1) == 1 and out.stride(1) == 1 and out.dtype == o.dtype
+    assert talk.dtype == torch.float32 and talk.shape == (n_head, n_head) and talk.is_contiguous()
+    assert out.shape == (rows, n_head * v_dim)
+    assert gate is None or (gate.dtype == o.dtype and gate.shape == out.shape and gate.stride(1) == 1)
+    st = kernels().cbis_mix_heads(_ptr(o), c_int(o.stride(0)), _ptr(talk), _ptr(gate), c_int(gate.stride(0) if gate is not None else 0),
+                                  _ptr(out), c_int(out.stride(0)), c_int(rows), c_int(n_head), c_int(n_kv_head), c_int(v_dim),
+                                  c_int(dtype_code(o.dtype)), _stream())
+    _check(st, "mix_heads", f"rows={rows} heads={n_head}/{n_kv_head} v_dim={v_dim}")
+
+
 def blend_rows(a, b, blend: float, out):
     """out = (1 - blend) a + blend b element by element (32-bit arithmetic, one rounding); ``[rows, n]`` of one type,
     views with unit column stride are fine."""
@@ -1145,25 +1193,32 @@ def ssm_scan(xbc, proj, dt_off, dt_bias, a_log, d_skip, state, seg_slot, cu_rows
 ROUTE_SCORE = {"sigmoid": 0, "softmax": 1}
 
 
-def route_topk(h, router, top, score, renormalize, ids, weights, renorm_eps: float = 0.0, weight_scale: float = 1.0):
+def route_topk(h, router, top, score, renormalize, ids, weights, renorm_eps: float = 0.0, weight_scale: float = 1.0,
+               correction=None, side=None):
     """Router logits ``h @ router^T`` in 32-bit, scores by ``score``, the ``top`` largest per row into ``ids``
     (int32 ``[rows, top]``) with their weights (float32; divided by their sum + ``renorm_eps`` with ``renormalize``;
-    then times ``weight_scale``)."""
-    _need_cuda(h, router, ids, weights)
+    then times ``weight_scale``).  ``correction`` (32-bit, one per expert) joins the scores for the choice alone, not the
+    weights.  ``side`` (32-bit ``[rows]``): the router's last row is no expert's; side takes the sigmoid of its logit."""
+    _need_cuda(h, router, ids, weights, correction, side)
     rows, W = h.shape
-    E = router.shape[0]
+    E = router.shape[0] - (1 if side is not None else 0)
+    assert correction is None or (correction.dtype == torch.float32 and correction.numel() == E and correction.is_contiguous())
+    assert side is None or (side.dtype == torch.float32 and side.numel() >= rows and side.is_contiguous())
     assert h.stride(1) == 1 and router.is_contiguous() and router.shape[1] == W and router.dtype == h.dtype
     assert ids.dtype == torch.int32 and weights.dtype == torch.float32 and ids.is_contiguous() and weights.is_contiguous()
     assert ids.shape == (rows, top) and weights.shape == (rows, top)
     st = kernels().cbis_route_topk(_ptr(h), c_int(h.stride(0)), _ptr(router), _ptr(ids), _ptr(weights), c_int(rows),
                                    c_int(W), c_int(E), c_int(top), c_int(ROUTE_SCORE[score]), c_int(1 if renormalize else 0),
-                                   c_int(dtype_code(h.dtype)), _stream(), c_float(renorm_eps), c_float(weight_scale))
+                                   c_int(dtype_code(h.dtype)), _stream(), c_float(renorm_eps), c_float(weight_scale),
+                                   _ptr(correction), _ptr(side))
     _check(st, "route_topk", f"rows={rows} experts={E} top={top}")
 
 
-def routed_gate_up(h, gate_up, ids, weights, act, weight_on_input, hidden):
+def routed_gate_up(h, gate_up, ids, weights, act, weight_on_input, hidden, limit: float = 0.0, beta: float = 1.0,
+                   shift: float = 0.0):
     """hidden[(row, choice)] = act(s * gate_e(h[row])) * (s * up_e(h[row])), e the choice's expert, s its weight if
-    the weight multiplies the expert's input, else 1.  ``gate_up`` ``[experts, 2 * inner, width]``."""
+    the weight multiplies the expert's input, else 1.  ``gate_up`` ``[experts, 2 * inner, width]``; a choice beyond the
+    experts is an identity expert and has no hidden row.  ``limit``, ``beta``, ``shift``: as in ``gate_mul``."""
     _need_cuda(h, gate_up, ids, weights, hidden)
     rows, W = h.shape
     E, F2, _ = gate_up.shape
@@ -1172,21 +1227,25 @@ def routed_gate_up(h, gate_up, ids, weights, act, weight_on_input, hidden):
     assert hidden.shape == (rows * top, F2 // 2) and hidden.dtype == h.dtype == gate_up.dtype
     st = kernels().cbis_routed_gate_up(_ptr(h), c_int(h.stride(0)), _ptr(gate_up), _ptr(ids), _ptr(weights), _ptr(hidden),
                                        c_int(rows), c_int(W), c_int(F2 // 2), c_int(top), c_int(ACT[act]),
-                                       c_int(1 if weight_on_input else 0), c_int(dtype_code(h.dtype)), _stream())
+                                       c_int(1 if weight_on_input else 0), c_int(dtype_code(h.dtype)), _stream(), c_int(E),
+                                       c_float(limit), c_float(beta), c_float(shift))
     _check(st, "routed_gate_up", f"rows={rows} width={W} inner={F2 // 2} top={top}")
 
 
-def routed_down(hidden, down, ids, weights, weight_on_input, out, accumulate=False):
+def routed_down(hidden, down, ids, weights, weight_on_input, out, accumulate=False, h=None):
     """out[row] = the sum over the row's choices of down_e(hidden[(row, choice)]) (times the choice's weight unless
-    it already multiplied the input); ``down`` ``[experts, width, inner]``; out 32-bit, added to with ``accumulate``."""
-    _need_cuda(hidden, down, ids, weights, out)
+    it already multiplied the input); ``down`` ``[experts, width, inner]``; out 32-bit, added to with ``accumulate``.
+    ``h``: the feed-forward's input rows; a choice beyond the experts is an identity expert and adds its weight times
+    the row (without ``h`` no choice may be one)."""
+    _need_cuda(hidden, down, ids, weights, out, h)
     E, W, F = down.shape
     rows, top = ids.shape
     assert hidden.is_contiguous() and hidden.shape == (rows * top, F) and down.is_contiguous() and hidden.dtype == down.dtype
     assert out.dtype == torch.float32 and out.shape == (rows, W) and out.stride(1) == 1
     st = kernels().cbis_routed_down(_ptr(hidden), _ptr(down), _ptr(ids), _ptr(weights), _ptr(out), c_int(out.stride(0)),
                                     c_int(rows), c_int(W), c_int(F), c_int(top), c_int(1 if weight_on_input else 0),
-                                    c_int(1 if accumulate else 0), c_int(dtype_code(hidden.dtype)), _stream())
+                                    c_int(1 if accumulate else 0), c_int(dtype_code(hidden.dtype)), _stream(),
+                                  c_int(E if h is not None else 2 ** 31 - 1), _ptr(h), c_int(h.stride(0) if h is not None else 0))
     _check(st, "routed_down", f"rows={rows} width={W} inner={F} top={top}")
 
 
@@ -1206,11 +1265,13 @@ def _routed_plan_ints(pairs: int, experts: int) -> int:
     return int(fn(c_int(pairs), c_int(experts)))
 
 
-def routed_tiles(h, gate_up, down, ids, weights, act, weight_on_input, out, accumulate=False):
+def routed_tiles(h, gate_up, down, ids, weights, act, weight_on_input, out, accumulate=False, identity: int = 0,
+                 limit: float = 0.0, beta: float = 1.0, shift: float = 0.0):
     """The routed feed-forward for many rows of bfloat16: the (row, choice) pairs are sorted by expert on the device, an
     expert's pairs run in tiles of 128 rows on the tensor cores (gate and up with the gated activation in one kernel,
     then down), and a row's choices are summed in their order.  ``out`` 32-bit ``[rows, width]``, overwritten or, with
-    ``accumulate``, added to.  Nothing is read back to the host: it can be captured."""
+    ``accumulate``, added to.  Nothing is read back to the host: it can be captured.  ``identity``: how many choices beyond
+    the experts are identity experts (the row itself times the weight); ``limit``, ``beta``, ``shift``: as in ``gate_mul``."""
     _need_cuda(h, gate_up, down, ids, weights, out)
     rows, W = h.shape
     E, F2, _ = gate_up.shape
@@ -1219,11 +1280,12 @@ def routed_tiles(h, gate_up, down, ids, weights, act, weight_on_input, out, accu
     assert out.dtype == torch.float32 and out.shape == (rows, W) and out.stride(1) == 1
     plan = torch.empty(int(_routed_plan_ints(rows * top, E)), dtype=torch.int32, device=h.device)
     hidden = torch.empty((rows * top, F), dtype=torch.bfloat16, device=h.device)
-    y = torch.empty((rows * top, W), dtype=torch.float32, device=h.device) if (top > 1 or accumulate) else None
+    y = torch.empty((rows * top, W), dtype=torch.float32, device=h.device) if (top > 1 or accumulate or identity) else None
     st = kernels().cbis_routed_tiles(_ptr(h), c_int(h.stride(0)), _ptr(gate_up), _ptr(down), _ptr(ids), _ptr(weights),
                                      _ptr(plan), _ptr(hidden), _ptr(y), _ptr(out), c_int(out.stride(0)), c_int(rows),
                                      c_int(W), c_int(F), c_int(E), c_int(top), c_int(ACT[act]),
-                                     c_int(1 if weight_on_input else 0), c_int(1 if accumulate else 0), _stream())
+                                     c_int(1 if weight_on_input else 0), c_int(1 if accumulate else 0), _stream(), c_int(identity),
+                                     c_float(limit), c_float(beta), c_float(shift))
     _check(st, "routed_tiles", f"rows={rows} width={W} inner={F} experts={E} top={top}", launches=4 if y is not None else 3)
 
 

@@ -44,6 +44,8 @@ class Layer:
         extra = {}
         if spec.residual_scale != 1.0 or self.side is not None:
             extra = {"residual_scale": spec.residual_scale, "side": self.side}
+        if spec.stream_scale != 1.0:
+            extra["stream_scale"] = spec.stream_scale
         self.block = make_block(spec.arrangement, self.mixer, self.feed_forward, self.norm_mixer,
                                 self.norm_feed_forward, self.post_norm_mixer, self.post_norm_feed_forward, **extra)
         self.norm_names = tuple(spec.norm_prefixes)

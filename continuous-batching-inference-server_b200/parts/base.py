@@ -33,11 +33,14 @@ class Delta:
     delta applies it in the same pass if it can (``Norm.takes_post``), else it is applied on its own
     (``settle_delta``).  ``scale``: a constant on everything that is added (after ``post``), for a block that
     multiplies its parts' results before they join the stream; applied by the norm that adds the delta
-    (``Norm.takes_scale``) or on its own."""
+    (``Norm.takes_scale``) or on its own.  ``onto``: (norm, alpha), for a block whose norm stands AFTER the addition: the
+    stream becomes norm(alpha * stream + what is added) instead of the bare sum; the norm that adds the delta does it in
+    the same pass (``Norm.takes_onto``), else it is done on its own."""
     value: torch.Tensor
     bias: Optional[torch.Tensor] = None
     post: Optional["Norm"] = None
     scale: float = 1.0
+    onto: Optional[Tuple["Norm", float]] = None
 
 
 @dataclass(frozen=True)
@@ -164,6 +167,7 @@ class FeedForward(Part):
 
 class Norm(Part):
     takes_scale = False        # whether ``forward`` applies a delta's ``scale`` itself, in its one pass
+    takes_onto = False         # whether ``forward`` makes the stream norm(alpha * stream + delta) itself (``Delta.onto``)
 
     def forward(self, ctx, x: torch.Tensor, delta: Optional[Delta], rows: Optional[torch.Tensor] = None,
                 out_dtype: Optional[torch.dtype] = None) -> torch.Tensor:
@@ -228,16 +232,35 @@ class Head(Part):
         raise NotImplementedError
 
 
-def settle_delta(ctx, norm: Norm, delta: Optional[Delta]) -> Optional[Delta]:
+def settle_delta(ctx, norm: Norm, delta: Optional[Delta], x: Optional[torch.Tensor] = None) -> Optional[Delta]:
     """What ``norm`` can add as it is: a delta whose own norm, or whose scale, ``norm`` does not apply in its pass gets
-    them here."""
+    them here.  A delta that changes the stream ``x`` by more than an addition (``onto``) is added here, in place, if
+    ``norm`` does not do that: nothing is left to add."""
     if delta is None:
+        return None
+    if delta.onto is not None and not norm.takes_onto:
+        add_onto(ctx, x, delta)
         return None
     if delta.post is not None and not norm.takes_post(delta.post):
         delta = Delta(delta.post.apply(ctx, delta.value, delta.bias), scale=delta.scale)
     if delta.scale != 1.0 and not norm.takes_scale:
         delta = plain_delta(ctx, delta)
     return delta
+
+
+def onto_args(delta: Optional[Delta]) -> dict:
+    """What ``ops.add_rmsnorm`` is told about a delta's ``onto``: nothing without one."""
+    if delta is None or delta.onto is None:
+        return {}
+    norm, alpha = delta.onto
+    return {"x_scale": alpha, "stream": norm.as_rmsnorm()}
+
+
+def add_onto(ctx, x: torch.Tensor, delta: Delta) -> None:
+    """x = norm(alpha * x + delta) in place, on its own, for a delta with ``onto``."""
+    from ..kernels import ops
+    rest = plain_delta(ctx, Delta(delta.value, delta.bias, delta.post, delta.scale))
+    ops.add_rmsnorm(x, rest.value, rest.bias, None, None, 0.0, 0.0, None, **onto_args(delta))
 
 
 def plain_delta(ctx, delta: Delta) -> Delta:

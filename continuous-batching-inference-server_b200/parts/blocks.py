@@ -7,13 +7,18 @@ import torch
 
 from ..kernels import ops
 from .attention import PagedAttention
-from .base import Block, Delta, plain_delta, register_block, settle_delta
+from .base import Block, Delta, add_onto, plain_delta, register_block, settle_delta
 from .dense import DenseFeedForward, NoFeedForward
 from .layernorm import LayerNorm, NoNorm
+from .rmsnorm import RMSNorm
 
 
 def _add_pending(ctx, x, d) -> None:
-    """x += what a layer left pending (through the delta's own norm first, if it names one)."""
+    """x += what a layer left pending (through the delta's own norm first, if it names one; x = norm(alpha x + that), if
+    that is what the layer wants)."""
+    if d.onto is not None:
+        add_onto(ctx, x, d)
+        return
     d = plain_delta(ctx, d)
     ops.add_delta(x, d.value, d.bias)
 
@@ -224,7 +229,35 @@ class ScaledPreNormBlock(Block):
         return d
 
 
+class PostNormBlock(Block):
+    """x = norm_1(alpha x + mixer(x)); x = norm_2(alpha x + feed_forward(x)): a norm AFTER every addition, and the parts
+    read the stream itself.  ``stream_scale`` alpha is a constant of the model.  A part's result is handed on with the
+    norm and the constant (``Delta.onto``): whoever reads the stream next (the next part, the final norm) adds it,
+    normalises the sum, keeps that as the stream (32-bit) and takes its own rows from it in ONE pass.  A part never adds
+    into the stream itself (the sum has to be scaled and normalised).  A layer without a feed-forward is the first half."""
+
+    def __init__(self, mixer, feed_forward, norm_mixer, norm_feed_forward, stream_scale: float = 1.0):
+        super().__init__(mixer, feed_forward, norm_mixer, norm_feed_forward)
+        self.stream_scale = float(stream_scale)
+        for n in (norm_mixer,) + (() if isinstance(feed_forward, NoFeedForward) else (norm_feed_forward,)):
+            if not isinstance(n, RMSNorm):
+                raise ValueError("a post-norm block takes root-mean-square norms")
+        self.as_it_is = NoNorm(norm_mixer.width)
+
+    def _after(self, d, norm):
+        return Delta(d.value, d.bias, d.post, d.scale, (norm, self.stream_scale))
+
+    def forward(self, ctx, x, pending, cache, state):
+        h = self.as_it_is.forward(ctx, x, pending)
+        d = self._after(self.mixer.forward(ctx, h, cache, state), self.norm_mixer)
+        if isinstance(self.feed_forward, NoFeedForward):
+            return d
+        h = self.as_it_is.forward(ctx, x, d)
+        return self._after(self.feed_forward.forward(ctx, h), self.norm_feed_forward)
+
+
 register_block("pre_norm", PreNormBlock)
+register_block("post_norm", PostNormBlock)
 register_block("pre_norm_scaled", ScaledPreNormBlock)
 register_block("parallel", ParallelBlock)
 register_block("sandwich", SandwichBlock)

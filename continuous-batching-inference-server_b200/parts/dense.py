@@ -72,16 +72,18 @@ class GatedFeedForward(FeedForward):
     """down(act(gate h) * (up h)): three matrices stored ``[out, in]``, no biases; the gate's and the up
     projection's rows form one matrix, so one product gives both, and the activation and the product of the two
     halves are taken in 32-bit and rounded once.  With ``biases`` each of the three has a bias (its matrix's name with
-    ``.b``), added to the 32-bit sums.  ``names``: what follows the layer's prefix in the names of the gate, up and
-    down matrices."""
+    ``.b``), added to the 32-bit sums.  ``limit`` > 0 cuts the gate's projection off at limit from above and the up
+    projection at -limit and limit; ``beta`` is silu's inner factor (g * sigmoid(beta g)); ``up_shift`` is added to the up
+    projection after the cut.  ``names``: what follows the layer's prefix in the names of the gate, up and down matrices."""
 
     def __init__(self, width: int, inner: int, activation: str = "silu", names=("mlp.gate", "mlp.up", "mlp.down"),
-                 biases: bool = False):
+                 biases: bool = False, limit: float = 0.0, beta: float = 1.0, up_shift: float = 0.0):
         if activation not in ops.ACT or not activation:
             raise ValueError(f"activation {activation!r} is not one of {sorted(k for k in ops.ACT if k)}")
         self.width, self.inner, self.activation = int(width), int(inner), activation
         self.gate_name, self.up_name, self.down_name = names
         self.biases = bool(biases)
+        self.shape = {"limit": float(limit), "beta": float(beta), "shift": float(up_shift)}      # of the gated product
         self.w_gate_up = self.w_down = self.b_gate_up = self.b_down = None
 
     def tensors(self, prefix):
@@ -106,11 +108,15 @@ class GatedFeedForward(FeedForward):
     def streamed_weights(self):
         return [self.w_gate_up, self.w_down]
 
-    def forward(self, ctx, h):
+    def _inside(self, h, row_gate=None):
         F = self.inner
         gu = ops.linear(h, self.w_gate_up, self.b_gate_up)
         a = torch.empty((h.shape[0], F), dtype=h.dtype, device=h.device)
-        ops.gate_mul(gu[:, :F], gu[:, F:], self.activation, a)
+        ops.gate_mul(gu[:, :F], gu[:, F:], self.activation, a, row_gate=row_gate, **self.shape)
+        return a
+
+    def forward(self, ctx, h):
+        a = self._inside(h)
         if self.b_down is None:
             if ops.linear_residual(a, self.w_down, ctx.residual):   # the product adds into the residual stream itself
                 return None
@@ -119,13 +125,10 @@ class GatedFeedForward(FeedForward):
             return None
         return Delta(ops.linear(a, self.w_down, None, None, out_dtype=torch.float32), self.b_down)
 
-
-    def forward_into(self, h, out) -> None:
-        """out += this feed-forward of h; ``out``: 32-bit rows (another part's result that this one joins)."""
-        F = self.inner
-        gu = ops.linear(h, self.w_gate_up, self.b_gate_up)
-        a = torch.empty((h.shape[0], F), dtype=h.dtype, device=h.device)
-        ops.gate_mul(gu[:, :F], gu[:, F:], self.activation, a)
+    def forward_into(self, h, out, row_gate=None) -> None:
+        """out += this feed-forward of h; ``out``: 32-bit rows (another part's result that this one joins).  ``row_gate``
+        (32-bit, one number per row) multiplies it (a feed-forward without a down bias)."""
+        a = self._inside(h, row_gate)
         if self.b_down is None and ops.linear_residual(a, self.w_down, out):
             return
         ops.add_delta(out, ops.linear(a, self.w_down, None, None, out_dtype=torch.float32), self.b_down)

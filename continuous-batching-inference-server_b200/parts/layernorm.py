@@ -7,7 +7,7 @@ import torch
 
 from ..kernels import ops
 from ..weights.loader import TensorDecl
-from .base import Delta, Norm, register_norm, settle_delta
+from .base import Delta, Norm, onto_args, register_norm, settle_delta
 
 
 class LayerNorm(Norm):
@@ -35,7 +35,7 @@ class LayerNorm(Norm):
 
     def forward(self, ctx, x, delta: Optional[Delta], rows=None, out_dtype=None):
         n = rows.shape[0] if rows is not None else x.shape[0]
-        delta = settle_delta(ctx, self, delta)
+        delta = settle_delta(ctx, self, delta, x)
         out = torch.empty((n, self.width), dtype=out_dtype or ctx.dtype, device=x.device)
         ops.add_layernorm(x, delta.value if delta else None, delta.bias if delta else None,
                           self.weight, self.bias, self.eps, out, rows)
@@ -61,14 +61,16 @@ class NoNorm(Norm):
     def takes_scale(self):
         return self.width <= ops.RMS_RESIDUAL_MAX_WIDTH
 
+    takes_onto = takes_scale
+
     def forward(self, ctx, x, delta: Optional[Delta], rows=None, out_dtype=None):
         n = rows.shape[0] if rows is not None else x.shape[0]
-        delta = settle_delta(ctx, self, delta)
+        delta = settle_delta(ctx, self, delta, x)
         out = torch.empty((n, self.width), dtype=out_dtype or ctx.dtype, device=x.device)
-        if delta is not None and (delta.post is not None or delta.scale != 1.0):
-            # x += post(delta) * scale; the rows go on as they are
+        if delta is not None and (delta.post is not None or delta.scale != 1.0 or delta.onto is not None):
+            # x += post(delta) * scale, or x = norm(alpha x + that); the rows go on as they are
             ops.add_rmsnorm(x, delta.value, delta.bias, delta.post.as_rmsnorm() if delta.post is not None else None,
-                            None, 0.0, 0.0, out, rows, delta_scale=delta.scale)
+                            None, 0.0, 0.0, out, rows, delta_scale=delta.scale, **onto_args(delta))
             return out
         ops.add_layernorm(x, delta.value if delta else None, delta.bias if delta else None, None, None, 0.0, out, rows)
         return out

@@ -7,7 +7,7 @@ import torch
 
 from ..kernels import ops
 from ..weights.loader import TensorDecl
-from .base import Delta, Norm, register_norm, settle_delta
+from .base import Delta, Norm, onto_args, register_norm, settle_delta
 
 
 class RMSNorm(Norm):
@@ -33,6 +33,7 @@ class RMSNorm(Norm):
         self.weight = self._vector(tensors[prefix + self.name], device)
 
     takes_scale = True
+    takes_onto = True
 
     def as_rmsnorm(self):
         return (self.weight, self.eps, self.offset) if self.weight is not None else None
@@ -42,13 +43,13 @@ class RMSNorm(Norm):
 
     def forward(self, ctx, x, delta: Optional[Delta], rows=None, out_dtype=None):
         n = rows.shape[0] if rows is not None else x.shape[0]
-        delta = settle_delta(ctx, self, delta)
+        delta = settle_delta(ctx, self, delta, x)
         out = torch.empty((n, self.width), dtype=out_dtype or ctx.dtype, device=x.device)
         post = None
         if delta is not None and delta.post is not None:
             post = (delta.post.weight, delta.post.eps, delta.post.offset)
         ops.add_rmsnorm(x, delta.value if delta else None, delta.bias if delta else None, post, self.weight, self.eps,
-                        self.offset, out, rows, delta_scale=delta.scale if delta else 1.0)
+                        self.offset, out, rows, delta_scale=delta.scale if delta else 1.0, **onto_args(delta))
         return out
 
     def apply(self, ctx, value, bias=None):
