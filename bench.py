@@ -115,7 +115,8 @@ def main() -> int:
     ap.add_argument("--steps", type=int, default=512)
     ap.add_argument("--warmup", type=int, default=16)
     ap.add_argument("--impl", default="b200", choices=["b200", "reference"])
-    ap.add_argument("--config", default="1.3b", choices=["1.3b", "6.7b", "xl", "batching", "vekedra", "figotar", "vatevik", "divitar"],
+    ap.add_argument("--config", default="1.3b", choices=["1.3b", "6.7b", "xl", "batching", "vekedra", "figotar", "vatevik", "divitar",
+                                                         "fororax"],
                     help="1.3b: the default measurement; 6.7b: batch-64 decode at context 2,048; "
                          "xl: 64 mixed requests through the scheduler (prompts 32-768, 256 outputs each); "
                          "batching: the reference's own workload at the reference's own sizes (both --impl arms); "
@@ -123,7 +124,8 @@ def main() -> int:
                          "of equal width and depth, and its own kernels one by one against their bytes; "
                          "figotar: the same for the Figotar design, beside Vekedra and the GPT-2 style model; "
                          "vatevik: the same for the Vatevik design, beside Figotar and the GPT-2 style model; "
-                         "divitar: the same for the Divitar design, beside Figotar, Vekedra and the GPT-2 style model")
+                         "divitar: the same for the Divitar design, beside Figotar, Vekedra and the GPT-2 style model; "
+                         "fororax: the same for the Fororax design, beside Divitar, Vatevik and the GPT-2 style model")
     ap.add_argument("--batch", type=int, default=None)
     ap.add_argument("--prompt-len", type=int, default=None)
     ap.add_argument("--layers", type=int, default=None, help="run fewer layers than the configuration has")
@@ -164,6 +166,8 @@ def main() -> int:
         return vatevik_workload(args, cb, torch)
     if args.config == "divitar":
         return divitar_workload(args, cb, torch)
+    if args.config == "fororax":
+        return fororax_workload(args, cb, torch)
     if args.config == "6.7b":
         args.skip_points = True
         args.batch = args.batch or 64
@@ -875,6 +879,238 @@ def divitar_kernels(torch, ops, pk):
             return lambda: ops.paged_decode_bf16(qkv, nh * hd, (nh + nkv) * hd, k, v, btB, row_seq, posB, slot_map, o, scratch,
                                                  counters, nh, nkv, hd, ps, hd ** -0.5, mask, ns)
         timed(decode, B * size * 2 * nkv * hd * 2, name)
+    return out
+
+
+def fororax_sizes(width, layers, positions=2048):
+    """A Fororax configuration with layers of the sizes a model of this width would have: attention with a logarithmic
+    distance bias and attention with mixed heads in turn (grouped key/value heads), every fourth layer reading the keys and
+    values of the layer two before it; every layer with routed experts (two of 16 or 8, and two identity outputs) and an
+    expert for all."""
+    big = width >= 2048
+    hd = 128 if big else 64
+    heads = width // hd
+    mix = {"dim": hd, "heads": heads, "kv_heads": max(1, heads // 4), "scale": hd ** -0.5, "vdim": hd}
+    moe = {"kind": "moe", "expert": {"ff": 11 * width // 16, "limit": 7.0},
+           "router": {"experts": 16 if big else 8, "identity": 2, "top": 2}, "shared": {"ff": 11 * width // 16, "limit": 7.0}}
+    out = []
+    for i in range(layers):
+        mixer = dict(mix)
+        if i % 4 == 2:
+            mixer["kv_from"] = i - 2
+        out.append({"type": ("attention", "attention_2")[i % 2], "mixer": mixer, "mlp": dict(moe)})
+    return {"architecture": "Fororax", "embedding": {"scale": 8.0}, "layers": out, "logit_softcap": 30.0,
+            "max_positions": positions, "norm": {"eps": 1e-6}, "postln_alpha": 2.0, "vocab": 32000, "width": width}
+
+
+def fororax_workload(args, cb, torch) -> int:
+    """Prefill (one 2,048-token prompt in one step) and decode (batch 8 from context 1,024, the captured step with
+    argmax on the device) of the Fororax design at two layer sizes, each beside Divitar (the closest model in its
+    feed-forwards: routed experts with one for all), Vatevik (the closest in its mixers: grouped heads with norms over q and
+    k and a sink) and the GPT-2 style model of equal width and depth; then the design's own kernels alone, at the larger
+    size, beside the like kernels of those models."""
+    from cbis_b200.kernels import ops
+    pk = peaks()
+    P, T, B = 2048, 2048, args.batch or 8
+    steps, warm = min(args.steps, 128), max(3, min(args.warmup, 8))
+    layers = args.layers or 8
+    gen = torch.Generator().manual_seed(0)
+    sampler = ClockSampler()
+    sampler.start()
+    sizes = {}
+    for width in (1024, 2048):
+        gpt = dict(architectures=["GPT2LMHeadModel"], model_type="gpt2", n_layer=layers, n_embd=width, n_head=16,
+                   n_inner=4 * width, vocab_size=32000, n_positions=P, activation_function="gelu",
+                   layer_norm_epsilon=1e-5, tie_word_embeddings=False)
+        sizes[f"width_{width}"] = {name: measure_model(args, cb, torch, pk, cfgd, 32000, B, P, T, steps, warm, gen)
+                                   for name, cfgd in (("fororax", fororax_sizes(width, layers, P)),
+                                                      ("divitar", divitar_sizes(width, layers)),
+                                                      ("vatevik", vatevik_sizes(width, layers)), ("gpt2_style", gpt))}
+    clocks = sampler.stop()
+    line = {"metric": f"Fororax prefill and decode tokens/s beside Divitar, Vatevik and the GPT-2 style model of equal "
+                      f"width and depth ({layers} layers, batch {B}, prompt {T})", "unit": "tokens/s", "n_gpus": 1,
+            "impl": "b200", "dtype": "bf16", "data": "synthetic (random weights, uniform random token ids)",
+            "higher_is_better": True, "value": sizes["width_2048"]["fororax"]["decode_tokens_per_s"], "sizes": sizes,
+            "kernels": fororax_kernels(torch, ops, pk), "clocks": clocks, "peaks": pk}
+    print(json.dumps(line))
+    return 0
+
+
+def fororax_kernels(torch, ops, pk):
+    """Microseconds of the kernels the design added or changed, alone, at the layer sizes of width 2,048, with the bytes
+    each has to move over its time as a fraction of the measured copy bandwidth (attention over prompts: its
+    arithmetic as a fraction of the measured bf16 peak), each beside the like kernel of the closest model at equal
+    sizes."""
+    bf = torch.bfloat16
+    out = {}
+    timed = graph_timer(torch, pk, out)
+    W, nh, nkv, hd = 2048, 16, 4, 128
+    E, top, F = 16, 2, 1408
+    dq, dk = nh * hd, nkv * hd
+    freqs = (10000.0 ** (-2.0 * torch.arange(hd // 2, dtype=torch.float64) / hd)).float().cuda()
+    wide = {"limit": 7.0, "beta": 1.702, "shift": 1.0}
+    for rows, segs, tag in ((2048, 1, "prefill_2048"), (8, 8, "decode_8")):
+        pos = torch.arange(rows, dtype=torch.int32, device="cuda")
+
+        def head_norm():
+            buf, w = torch.randn(rows, dq + 2 * dk, device="cuda").to(bf), torch.ones(hd, device="cuda")
+            return lambda: ops.qk_head_norm(buf, 0, nh, dq, nkv, hd, w, w, 1e-6)
+        timed(head_norm, rows * 2 * (dq + dk) * 2, f"qk_head_norm_{tag}")
+
+        def whole_norm():       # Vatevik's: one norm over all of q and one over all of k, rotated
+            buf = torch.randn(rows, dq + 2 * dk, device="cuda").to(bf)
+            wq, wk = torch.ones(dq, device="cuda"), torch.ones(dk, device="cuda")
+            return lambda: ops.qk_prepare(buf, 0, nh, dq, nkv, hd, wq, wk, 1e-6, pos, freqs, hd)
+        timed(whole_norm, rows * 2 * (dq + dk) * 2, f"closest_model_qk_prepare_{tag}")
+
+        def post_norm(w_out):
+            def make():
+                x, d = torch.randn(rows, W, device="cuda"), torch.randn(rows, W, device="cuda")
+                w, ws = torch.ones(W, device="cuda"), torch.ones(W, device="cuda")
+                o = torch.empty(rows, W, dtype=bf, device="cuda")
+                return lambda: ops.add_rmsnorm(x, d, None, None, w if w_out else None, 1e-6, 0.0, o, x_scale=2.0, stream=(ws, 1e-6, 0.0))
+            return make
+        timed(post_norm(False), rows * W * (4 + 4 + 4 + 2), f"add_rmsnorm_of_the_sum_{tag}")
+        timed(post_norm(True), rows * W * (4 + 4 + 4 + 2), f"add_rmsnorm_of_the_sum_then_a_norm_{tag}")
+
+        def pre_norm():
+            x, d = torch.randn(rows, W, device="cuda"), torch.randn(rows, W, device="cuda")
+            w = torch.ones(W, device="cuda")
+            o = torch.empty(rows, W, dtype=bf, device="cuda")
+            return lambda: ops.add_rmsnorm(x, d, None, None, w, 1e-6, 0.0, o, delta_scale=0.5)
+        timed(pre_norm, rows * W * (4 + 4 + 4 + 2), f"closest_model_add_rmsnorm_{tag}")
+
+        def route(new):
+            def make():
+                h = torch.randn(rows, W, device="cuda").to(bf)
+                r = torch.randn(E + (3 if new else 0), W, device="cuda").to(bf)
+                ids = torch.empty(rows, top, dtype=torch.int32, device="cuda")
+                wt, side = torch.empty(rows, top, device="cuda"), torch.empty(rows, device="cuda")
+                corr = torch.zeros(E + 2, device="cuda")
+                if new:
+                    return lambda: ops.route_topk(h, r, top, "softmax", False, ids, wt, correction=corr, side=side)
+                return lambda: ops.route_topk(h, r, top, "sigmoid", True, ids, wt, 1e-20, 2.5)
+            return make
+        timed(route(True), rows * W * 2 + (E + 3) * W * 2, f"route_topk_corrected_with_a_row_gate_{tag}")
+        timed(route(False), rows * W * 2 + E * W * 2, f"closest_model_route_topk_{tag}")
+
+        def experts(new):
+            def make():
+                h = torch.randn(rows, W, device="cuda").to(bf)
+                gu = (torch.randn(E, 2 * F, W, device="cuda") * 0.02).to(bf)
+                dn = (torch.randn(E, W, F, device="cuda") * 0.02).to(bf)
+                g = torch.Generator().manual_seed(1)
+                ids = torch.randint(0, E + (2 if new else 0), (rows, top), generator=g).int().cuda()
+                wt = torch.rand(rows, top, generator=g).cuda()
+                hid = torch.empty(rows * top, F, dtype=bf, device="cuda")
+                o = torch.empty(rows, W, device="cuda")
+                kw = wide if new else {}
+
+                def run():
+                    if ops.routed_tiles_takes(h, gu, dn):          # as the part chooses
+                        ops.routed_tiles(h, gu, dn, ids, wt, "silu", False, o, identity=2 if new else 0, **kw)
+                    else:
+                        ops.routed_gate_up(h, gu, ids, wt, "silu", False, hid, **kw)
+                        ops.routed_down(hid, dn, ids, wt, False, o, h=h if new else None)
+                return run
+            return make
+        for new, name in ((True, "routed_feed_forward_with_identity_experts"), (False, "closest_model_routed_feed_forward")):
+            share = E / (E + 2) if new else 1.0          # of the choices, those that are experts
+            touched = min(E, round(rows * top * share))
+            timed(experts(new), touched * 3 * F * W * 2 + rows * W * 6, f"{name}_{tag}", copies=2,
+                  flops=2.0 * rows * top * share * 3 * F * W)
+
+        def gated(new):
+            def make():
+                gu = torch.randn(rows, 2 * F, device="cuda").to(bf)
+                a = torch.empty(rows, F, dtype=bf, device="cuda")
+                rg = torch.rand(rows, device="cuda")
+                kw = dict(wide, row_gate=rg) if new else {}
+                return lambda: ops.gate_mul(gu[:, :F], gu[:, F:], "silu", a, **kw)
+            return make
+        timed(gated(True), rows * F * 3 * 2, f"gate_mul_cut_off_with_a_row_gate_{tag}")
+        timed(gated(False), rows * F * 3 * 2, f"closest_model_gate_mul_{tag}")
+
+        def mix():
+            o = torch.randn(rows, nh * nkv * hd, device="cuda").to(bf)
+            t = torch.randn(nh, nh, device="cuda")
+            gate = torch.randn(rows, dq, device="cuda").to(bf)
+            r = torch.empty(rows, dq, dtype=bf, device="cuda")
+            return lambda: ops.mix_heads(o, t, nh, nkv, hd, r, gate)
+        timed(mix, rows * (nh * nkv * hd + 2 * dq) * 2, f"mix_heads_{tag}")
+
+    # attention of 16 query heads over 4 key/value heads of 128 over a prompt of 2,048 and for 8 decoding rows behind 2,047
+    # keys; pages of 16
+    ps, ctx_len = 16, 2048
+    pages = ctx_len // ps
+    bt1 = torch.arange(pages, dtype=torch.int32, device="cuda").view(1, pages)
+    cu1 = torch.tensor([0, ctx_len], dtype=torch.int32, device="cuda")
+    zero1 = torch.zeros(1, dtype=torch.int32, device="cuda")
+    flops = 4.0 * ctx_len * (ctx_len + 1) / 2 * nh * hd
+    per_head = [torch.full((nh,), v, device="cuda") for v in (1.2, 0.3, 1.0)]
+    every = torch.zeros(nh * nkv, device="cuda")
+    talk = torch.randn(nh, nh, device="cuda") * 0.3
+
+    def prefill(kernel, v_heads=1, **kw):
+        def make():
+            q = torch.randn(ctx_len, nh * hd, device="cuda").to(bf)
+            k, v = (torch.randn(pages, nkv, ps, hd, device="cuda").to(bf) for _ in range(2))
+            o = torch.empty(ctx_len, nh * v_heads * hd, dtype=bf, device="cuda")
+            r = torch.empty(ctx_len, nh * hd, dtype=bf, device="cuda")
+
+            def run():
+                kernel(q, k, v, bt1, cu1, zero1, o, 0, 1, ctx_len, nh * v_heads, nkv, hd, ps, hd ** -0.5, 0,
+                       v_heads=v_heads, **kw)
+                if v_heads > 1:
+                    ops.mix_heads(o, talk, nh, nkv, hd, r)
+            return run
+        return make
+    slopes, rates, sinks = per_head
+    nbytes = ctx_len * (2 * nh + 2 * nkv) * hd * 2
+    timed(prefill(ops.paged_prefill_tc5, slopes=slopes, rates=rates), nbytes, "attention_prefill_2048_log_bias", flops=flops)
+    timed(prefill(ops.paged_prefill_bf16, slopes=slopes, rates=rates), nbytes, "attention_prefill_2048_log_bias_mma_sync_tiles", flops=flops)
+    timed(prefill(ops.paged_prefill_bf16, slopes=slopes, v_head_dim=hd), nbytes, "closest_model_attention_prefill_2048_linear_bias", flops=flops)
+    timed(prefill(ops.paged_prefill_tc5), nbytes, "attention_prefill_2048_plain", flops=flops)
+    timed(prefill(ops.paged_prefill_tc5, v_heads=nkv, sinks=every), nbytes, "attention_prefill_2048_mixed_heads_with_the_mixing", flops=flops)
+    timed(prefill(ops.paged_prefill_bf16, v_heads=nkv, sinks=every), nbytes, "attention_prefill_2048_mixed_heads_mma_sync_tiles", flops=flops)
+    timed(prefill(ops.paged_prefill_tc5, sinks=sinks), nbytes, "attention_prefill_2048_sink", flops=flops)
+    timed(prefill(ops.paged_prefill_bf16, sinks=sinks), nbytes, "closest_model_attention_prefill_2048_sink", flops=flops)
+    B = 8
+    btB = torch.arange(B * pages, dtype=torch.int32, device="cuda").view(B, pages)
+    row_seq = torch.arange(B, dtype=torch.int32, device="cuda")
+    posB = torch.full((B,), ctx_len - 1, dtype=torch.int32, device="cuda")
+    slot_map = (btB[:, -1] * ps + ps - 1).contiguous()
+
+    def decode(v_heads=1, mixing=False, **kw):
+        def make():
+            qkv = torch.randn(B, (nh + 2 * nkv) * hd, device="cuda").to(bf)
+            k, v = (torch.randn(B * pages, nkv, ps, hd, device="cuda").to(bf) for _ in range(2))
+            o = torch.empty(B, nh * v_heads * hd, dtype=bf, device="cuda")
+            r = torch.empty(B, nh * hd, dtype=bf, device="cuda")
+            if mixing:
+                blocks = ops.decode_mix_blocks(nh, nkv)
+                ns = ops.decode_splits(B, blocks, ctx_len)
+                scratch = torch.empty(ops.decode_mix_scratch_floats(B, nh, hd, ctx_len, ns), device="cuda")
+                counters = torch.zeros(B * blocks, dtype=torch.int32, device="cuda")
+                return lambda: ops.decode_mix_bf16(qkv, nh * hd, (nh + nkv) * hd, k, v, btB, row_seq, posB, slot_map, talk, sinks,
+                                                   None, r, scratch, counters, ctx_len, nh, nkv, hd, hd, ps, hd ** -0.5, 0, ns)
+            ns = ops.decode_splits(B, nh * v_heads, ctx_len)
+            scratch = torch.empty(max(1, ops.decode_scratch_floats(B, nh * v_heads, hd, ns)), device="cuda")
+            counters = torch.zeros(B * nh * v_heads, dtype=torch.int32, device="cuda")
+
+            def run():
+                ops.paged_decode_bf16(qkv, nh * hd, (nh + nkv) * hd, k, v, btB, row_seq, posB, slot_map, o, scratch, counters,
+                                      nh * v_heads, nkv, hd, ps, hd ** -0.5, 0, ns, v_heads=v_heads, **kw)
+                if v_heads > 1:
+                    ops.mix_heads(o, talk, nh, nkv, hd, r)
+            return run
+        return make
+    nbytes = B * ctx_len * 2 * nkv * hd * 2
+    timed(decode(slopes=slopes, rates=rates), nbytes, "attention_decode_8_log_bias")
+    timed(decode(slopes=slopes), nbytes, "closest_model_attention_decode_8_linear_bias")
+    timed(decode(mixing=True), nbytes, "attention_decode_8_mixed_heads")
+    timed(decode(v_heads=nkv, sinks=every), nbytes, "attention_decode_8_mixed_heads_every_head_over_every_value_head")
+    timed(decode(sinks=sinks), nbytes, "closest_model_attention_decode_8_sink")
     return out
 
 

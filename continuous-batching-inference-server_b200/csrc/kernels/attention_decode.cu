@@ -243,18 +243,19 @@ paged_decode_bf16_kernel(const __nv_bfloat16* qkv, int ld, int k_off, int v_off,
 // The fast form for head sizes 64 and 128 and pages of a multiple of 16 keys: decode_tc_item of
 // attention_decode_tc.cuh, one block of four warps per (row, head, split).
 // ---------------------------------------------------------------------------------------------
-template <int HD>
+template <int HD, bool BIAS>
 __global__ void __launch_bounds__(DEC_WARPS * 32, 4)   // 128 registers: four blocks per SM
 paged_decode_tc_kernel(const __nv_bfloat16* qkv, int ld, int k_off, int v_off, __nv_bfloat16* kc, __nv_bfloat16* vc,
                        const int* block_table, int max_blocks, const int* row_seq, const int* positions,
                        const int* slot_mapping, __nv_bfloat16* __restrict__ out, int out_ld, float* part,
                        unsigned int* counters, int n_head, int n_kv_head, int ps, float scale, int window,
-                       int nsplit, const float* __restrict__ sinks) {
+                       int nsplit, const float* __restrict__ sinks, const float* __restrict__ slopes,
+                       const float* __restrict__ rates) {
   __shared__ DecodeTcShared<HD> sm;
   pdl_trigger();
-  decode_tc_item<HD, true, (HD <= 64 ? 2 : 1)>(qkv, ld, k_off, v_off, kc, vc, block_table, max_blocks, row_seq, positions, slot_mapping, out,
+  decode_tc_item<HD, true, (HD <= 64 ? 2 : 1), BIAS>(qkv, ld, k_off, v_off, kc, vc, block_table, max_blocks, row_seq, positions, slot_mapping, out,
                            out_ld, part, counters, n_head, n_kv_head, ps, scale, window, nsplit, blockIdx.x, blockIdx.y,
-                           blockIdx.z, threadIdx.x, sm, 0, sinks);
+                           blockIdx.z, threadIdx.x, sm, 0, sinks, slopes, rates);
 }
 
 // After a decode step whose next tokens were chosen on the device: the chosen token becomes the
@@ -312,10 +313,10 @@ CBIS_EXPORT int cbis_paged_decode_bf16(const void* qkv, int ld, int k_off, int v
                                        int temp_every, const float* rates, int v_heads) {
   if (rows <= 0) return CBIS_OK;
   // hdv (0: the keys' width, values in pages of their own): the values' width.  With values of another width or in
-  // the keys' rows, a bias or a temperature the lane-group form runs whatever the head size; a sink alone is
-  // taken by both forms (it joins the denominator where the parts are merged)
+  // the keys' rows, a linear bias or a temperature the lane-group form runs whatever the head size; a sink (it joins
+  // the denominator where the parts are merged) and a bias that grows with the logarithm are taken by both forms
   if (hdv <= 0) hdv = hd, v_row = hd;
-  const bool extended = hdv != hd || v_row != hd || slopes || temp_every > 0 || v_heads > 1;
+  const bool extended = hdv != hd || v_row != hd || (slopes && !rates) || temp_every > 0 || v_heads > 1;
   if (v_heads != 1 && (v_heads != n_kv_head || n_head % v_heads)) return CBIS_ERR_BAD_SIZE;
   if (hdv > 256 || hdv % 8 || v_row < hdv || v_row % 8) return CBIS_ERR_BAD_SIZE;
   if (hd <= 0 || hd > 256 || hd % 8 || ps <= 0 || n_head <= 0 || n_kv_head <= 0 || (n_head / v_heads) % n_kv_head || nsplit < 1 || nsplit > 32)
@@ -329,17 +330,12 @@ CBIS_EXPORT int cbis_paged_decode_bf16(const void* qkv, int ld, int k_off, int v
   const int chunks = (hd > hdv ? hd : hdv) / 8;
   cudaError_t e;
   if ((hd == 64 || hd == 128) && ps % 16 == 0 && !extended) {
-    if (hd == 128)
-      e = launch_pdl(paged_decode_tc_kernel<128>, grid, dim3(DEC_WARPS * 32), 0, st, (const __nv_bfloat16*)qkv, ld, k_off,
+    auto kern = hd == 128 ? (slopes ? paged_decode_tc_kernel<128, true> : paged_decode_tc_kernel<128, false>)
+                          : (slopes ? paged_decode_tc_kernel<64, true> : paged_decode_tc_kernel<64, false>);
+    return (int)launch_pdl(kern, grid, dim3(DEC_WARPS * 32), 0, st, (const __nv_bfloat16*)qkv, ld, k_off,
                      v_off, (__nv_bfloat16*)kc, (__nv_bfloat16*)vc, block_table, max_blocks, row_seq, positions,
                      slot_mapping, (__nv_bfloat16*)out, out_ld, part, counters, n_head, n_kv_head, ps, scale, window,
-                     nsplit, sinks);
-    else
-      e = launch_pdl(paged_decode_tc_kernel<64>, grid, dim3(DEC_WARPS * 32), 0, st, (const __nv_bfloat16*)qkv, ld, k_off,
-                     v_off, (__nv_bfloat16*)kc, (__nv_bfloat16*)vc, block_table, max_blocks, row_seq, positions,
-                     slot_mapping, (__nv_bfloat16*)out, out_ld, part, counters, n_head, n_kv_head, ps, scale, window,
-                     nsplit, sinks);
-    return (int)e;
+                     nsplit, sinks, slopes, rates);
   }
 #define CBIS_DEC(LPK)                                                                                             \
   e = launch_pdl(paged_decode_bf16_kernel<LPK>, grid, dim3(DEC_WARPS * 32), 0, st, (const __nv_bfloat16*)qkv, ld, \

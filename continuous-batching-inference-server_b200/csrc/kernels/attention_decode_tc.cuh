@@ -77,14 +77,16 @@ struct DecodeTcShared {
 // hardware barrier the group meets at.  STANDALONE: the group is a block launched for this alone, which waits for
 // the kernels ahead (programmatic dependent launch) after it has fetched what they do not write.  The group's
 // threads must have met (group_sync) between two calls, since the calls share `sm`.
-template <int HD, bool STANDALONE, int TPW = 1>
+template <int HD, bool STANDALONE, int TPW = 1, bool BIAS = false>
 __device__ __forceinline__ void decode_tc_item(const __nv_bfloat16* qkv, int ld, int k_off, int v_off, __nv_bfloat16* kc,
                                                __nv_bfloat16* vc, const int* block_table, int max_blocks,
                                                const int* row_seq, const int* positions, const int* slot_mapping,
                                                __nv_bfloat16* out, int out_ld, float* part, unsigned int* counters,
                                                int n_head, int n_kv_head, int ps, float scale, int window, int nsplit,
                                                int row, int h, int split, int tid, DecodeTcShared<HD>& sm, int bar,
-                                               const float* __restrict__ sinks = nullptr) {
+                                               const float* __restrict__ sinks = nullptr,
+                                               const float* __restrict__ slopes = nullptr,
+                                               const float* __restrict__ rates = nullptr) {
   constexpr int NC = HD / 32;        // 16-byte loads per key for the score fragments (4 lanes x 16 B = 32 dims each)
   constexpr int LPK = HD / 8;        // lanes per key in the coalesced V loads
   constexpr int KPL = 32 / LPK;      // keys per warp-wide V load
@@ -181,6 +183,12 @@ __device__ __forceinline__ void decode_tc_item(const __nv_bfloat16* qkv, int ld,
   // A round: the values of this round's tiles are asked for, the scores are taken from the keys (asked for a round
   // earlier), the keys of the next round are asked for, and the softmax update and P V of this round run while they
   // come: a warp has loads on their way nearly all the time, not only while it waits for them.
+  float slope = 0.f;                                 // BIAS: a distance bias, taken off the scaled score
+  const float* rate = nullptr;
+  if constexpr (BIAS) {
+    slope = slopes[h];
+    rate = rates ? rates + h : nullptr;
+  }
   bool have_keys = preloaded, have_values = preloaded;
   for (; (tile << 4) < ke; tile += DEC_WARPS * TPW) {
     if (!have_keys) load_keys(tile);
@@ -208,6 +216,7 @@ __device__ __forceinline__ void decode_tc_item(const __nv_bfloat16* qkv, int ld,
       for (int e = 0; e < 4; ++e) {
         const int j = j0 + (e >> 1) * 8 + 2 * t + (e & 1);
         s4[u][e] = (g == 0 && j >= kstart && j < ke) ? sc[e >> 1][e & 1] * scale : -INFINITY;
+        if (BIAS && g == 0) s4[u][e] -= distance_bias(slope, rate, (float)max(pos - j, 0));
         mx = fmaxf(mx, s4[u][e]);
       }
     }

@@ -24,6 +24,12 @@
 // Shared memory (113 KB) and tensor memory (256 of 512 columns) are sized for TWO blocks per SM: while
 // one block's softmax warps work, the other's products run.
 //
+// A sink per head joins the denominator where the two blocks' parts meet.  A head's distance bias slope * ln(1 + rate *
+// distance) (BIAS) is taken from a table in shared memory of the 191 distances between the tile's rows and keys: the
+// softmax threads make it while the scores are still being computed (one or two logarithms a thread and tile instead of
+// 64), and a thread reads its row's 64 entries without conflicts.  With v_heads > 1 every query head attends to the values of every key/value
+// head (head_place in common.cuh).
+//
 // Every wait on an mbarrier is bounded; when a limit runs out the block sets *error, stops, frees its
 // tensor memory and returns (its output rows are then invalid, and the host raises).
 #include "attention_merge.cuh"
@@ -42,6 +48,7 @@ constexpr int P_BYTES = BM * 128;              // 128 rows of 64 keys
 constexpr int STAGES = 2;
 // Q, keys (one stage), values (STAGES), P (two buffers), barriers; HD: the head size, 64 or 128
 constexpr int smem_bytes(int HD) { return (HD / 64) * (Q_HALF_BYTES + (1 + STAGES) * KV_HALF_BYTES) + 2 * P_BYTES + 128; }
+constexpr int TABLE = BM + BN;                  // entries of the distance bias's table (191 in use)
 constexpr float RAISE_BY = 8.f;                // the reference is raised when a tile's maximum exceeds it by 2^8
 constexpr int THREADS = 224;                   // warp 0: Q and keys, warp 1: MMA + tensor memory, warps 2..5: softmax, warp 6: values
 constexpr unsigned SPIN_LIMIT = 1u << 21;      // tries of up to 1 us each
@@ -156,17 +163,24 @@ __device__ __forceinline__ void tmem_st32(unsigned taddr, const float* v) {
   asm volatile("tcgen05.wait::st.sync.aligned;" ::: "memory");
 }
 
+// The 128 softmax threads (warps 2..5) meet at a barrier of their own.
+__device__ __forceinline__ void softmax_warps_meet() {
+  __syncwarp();
+  asm volatile("bar.sync 1, 128;" ::: "memory");
+}
+
 // grid: row tiles of the longest segment x heads x segments from seg0 on, in one dimension, times two: the two
 // blocks of a cluster share a row tile, the first takes the first half of its key tiles and the second the rest,
 // and at the end the second hands its sum, reference and output to the first through distributed shared memory.
 // The row tile with the most keys decides how long the kernel runs, and its chain of tiles is halved this way.
-template <int HD>
+template <int HD, bool BIAS>
 __global__ void __cluster_dims__(2, 1, 1) __launch_bounds__(THREADS, 2)
 paged_prefill_tc5_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                          const __grid_constant__ CUtensorMap map_v, const int* block_table, int max_blocks,
                          const int* cu_rows, const int* seg_start, __nv_bfloat16* out, int out_ld, int seg0, int n_seg,
                          int n_head, int n_kv_head, int ps, float scale_log2e, int window, int n_chunks, int chunk_keys,
-                         float* partial, int row0, int* error) {
+                         float* partial, int row0, int* error, const float* __restrict__ sinks,
+                         const float* __restrict__ slopes, const float* __restrict__ rates, int v_heads) {
   constexpr int HALVES = HD / 64, Q_BYTES = HALVES * Q_HALF_BYTES, KV_BYTES = HALVES * KV_HALF_BYTES;
   extern __shared__ __align__(1024) unsigned char base[];   // no byte to spare for rounding the address up: checked below
   unsigned char* sQ = base;                                   // 2 halves of the head dim
@@ -180,6 +194,7 @@ paged_prefill_tc5_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
                      *s_full = bars + 9, *p_ready = bars + 11, *pv_done = bars + 13;   // k_full/k_empty: [0] only; p_ready, pv_done: [2], tiles in turn
   unsigned* tmem_slot = reinterpret_cast<unsigned*>(bars + 15);
   volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_slot + 1);
+  float* table = reinterpret_cast<float*>(sP + 2 * P_BYTES + 128);      // BIAS: entry e holds the bias (log2 units) of distance pos0 - j0 - (BN - 1) + e
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   // late row tiles have the most keys to walk: blocks are numbered so that those of ALL heads and segments come
@@ -195,7 +210,7 @@ paged_prefill_tc5_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
     if (threadIdx.x == 0) atomicExch(error, 18);
     return;
   }
-  const int hk = h / (n_head / n_kv_head);
+  const HeadPlace hp = head_place(h, n_head, n_kv_head, v_heads);
   const int pos0 = seg_start[seg] + tile * BM;
   const int rows_here = min(BM, n_rows - tile * BM);
   int kend = pos0 + rows_here;
@@ -261,7 +276,7 @@ paged_prefill_tc5_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
       bar_expect(q_full, Q_BYTES);
       const int qrow = r_begin + tile * BM;
 #pragma unroll
-      for (int hh = 0; hh < HALVES; ++hh) tma_2d(sQ + hh * Q_HALF_BYTES, &map_q, h * HD + hh * 64, qrow, q_full);
+      for (int hh = 0; hh < HALVES; ++hh) tma_2d(sQ + hh * Q_HALF_BYTES, &map_q, hp.query * HD + hh * 64, qrow, q_full);
     }
     const int piece = min(ps, BN), pieces_per_tile = BN / piece, piece_shift = 31 - __clz(piece);
     // copies tile j's keys (kv = 0) or values (kv = 1) into their stage; false when the block has given up
@@ -285,7 +300,7 @@ paged_prefill_tc5_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
       stop = __shfl_sync(0xffffffffu, stop, 0);
       if (stop) return false;
       if (mine) {
-        const int grow = (page * n_kv_head + hk) * ps + j0 % ps;   // row of the run's first key in the [rows, HD] view
+        const int grow = (page * n_kv_head + (kv ? hp.value : hp.key)) * ps + j0 % ps;   // row of the run's first key in the [rows, HD] view
         unsigned char* d = (kv ? sV : sK) + s * KV_BYTES + p0 * 128;
 #pragma unroll
         for (int hh = 0; hh < HALVES; ++hh) tma_2d(d + hh * KV_HALF_BYTES, kv ? &map_v : &map_k, hh * 64, grow, full);
@@ -355,13 +370,33 @@ paged_prefill_tc5_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
     // With the output in tensor memory a thread's share of a tile is one load of 64 scores, their maximum, 64
     // exponentials and eight 16-byte stores of P: no exchange between threads anywhere.
     const int p = pos0 + r;                         // this row's position
+    // a row that gives up leaves the loop, or, where the warps meet in every tile, goes on to the next meeting
+#define TC5_STOP { if constexpr (BIAS) continue; else break; }
+    float slope2 = 0.f, rate = 0.f;
+    if constexpr (BIAS) {
+      slope2 = slopes[h];                           // slope * ln(x) in log2 units is slope * log2(x)
+      rate = rates[h];
+    }
     for (int j = 0; j < n_tiles; ++j) {
       const int j0 = (kt_first + j) * BN;
-      if (!bar_wait(&s_full[j & 1], (j >> 1) & 1)) { atomicExch(error, 15); ok = false; break; }
-      if (*abort_flag) { ok = false; break; }
+      if constexpr (BIAS) {
+        // the four warps meet before the table is overwritten and when it is done; a row that has given up goes on
+        // meeting the others
+        const int low = pos0 - j0 - (BN - 1);
+        softmax_warps_meet();
+        for (int e = r; e < TABLE - 1; e += 128) table[e] = slope2 * log2f(fmaf(rate, (float)max(low + e, 0), 1.f));
+        softmax_warps_meet();
+        if (!ok) continue;
+      }
+      if (!bar_wait(&s_full[j & 1], (j >> 1) & 1)) { atomicExch(error, 15); ok = false; TC5_STOP }
+      if (*abort_flag) { ok = false; TC5_STOP }
       asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
       float v[BN];
       tmem_ld64(tmem_s + (j & 1) * BN + lane_addr, v);
+      if constexpr (BIAS) {      // from here on v is in log2 units with the bias taken off
+#pragma unroll
+        for (int i = 0; i < BN; ++i) v[i] = fmaf(v[i], scale_log2e, -table[r + BN - 1 - i]);
+      }
       const bool edge = (j0 + BN - 1 > pos0) || (window != 0 && j0 < first_seen(pos0 + BM - 1, window)) || j0 + BN > kend;
       if (edge) {
         // keys this row may see in this tile: [lo, hi), as columns of the tile
@@ -380,14 +415,14 @@ paged_prefill_tc5_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
         mx2 = fmaxf(mx2, v[i + 2]);
         mx3 = fmaxf(mx3, v[i + 3]);
       }
-      const float m_tile = fmaxf(fmaxf(mx0, mx1), fmaxf(mx2, mx3)) * scale_log2e;
+      const float m_tile = fmaxf(fmaxf(mx0, mx1), fmaxf(mx2, mx3)) * (BIAS ? 1.f : scale_log2e);
       // this tile's buffer of P was read by the products of the tile before the last
-      if (j > 1 && !bar_wait(&pv_done[j & 1], ((j - 2) >> 1) & 1)) { atomicExch(error, 16); ok = false; break; }
+      if (j > 1 && !bar_wait(&pv_done[j & 1], ((j - 2) >> 1) & 1)) { atomicExch(error, 16); ok = false; TC5_STOP }
       const bool raise = m_tile > m + RAISE_BY || (m == -INFINITY && m_tile > m);
       if (j > 0 && __any_sync(0xffffffffu, raise)) {
         // rescale the row of O in tensor memory; rows that keep their reference multiply by 1.  Only here does the
         // softmax wait for the products of the tile before, which write O.
-        if (!bar_wait(&pv_done[(j - 1) & 1], ((j - 1) >> 1) & 1)) { atomicExch(error, 16); ok = false; break; }
+        if (!bar_wait(&pv_done[(j - 1) & 1], ((j - 1) >> 1) & 1)) { atomicExch(error, 16); ok = false; TC5_STOP }
         asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
         const float f = raise ? exp2f(m - m_tile) : 1.f;
 #pragma unroll 1
@@ -410,7 +445,8 @@ paged_prefill_tc5_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
         unsigned pk[4];
 #pragma unroll
         for (int i = 0; i < 4; ++i) {
-          const float e0 = exp2f(fmaf(v[q8 * 8 + 2 * i], scale_log2e, -ref)), e1 = exp2f(fmaf(v[q8 * 8 + 2 * i + 1], scale_log2e, -ref));
+          const float e0 = exp2f(BIAS ? v[q8 * 8 + 2 * i] - ref : fmaf(v[q8 * 8 + 2 * i], scale_log2e, -ref)),
+                      e1 = exp2f(BIAS ? v[q8 * 8 + 2 * i + 1] - ref : fmaf(v[q8 * 8 + 2 * i + 1], scale_log2e, -ref));
           psum += e0;
           psum1 += e1;
           __nv_bfloat162 b2 = __floats2bfloat162_rn(e0, e1);
@@ -422,7 +458,7 @@ paged_prefill_tc5_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
       if (j0 + BN > kend && r < BN && j0 + r >= kend) {
         // the last tile: values of keys past the end are whatever the page held; P is zero there, but zero
         // times a NaN left by an earlier owner of the page would still be NaN: this thread clears key row r
-        if (!bar_wait(&v_full[j % STAGES], (j / STAGES) & 1)) { atomicExch(error, 13); ok = false; break; }   // they have landed
+        if (!bar_wait(&v_full[j % STAGES], (j / STAGES) & 1)) { atomicExch(error, 13); ok = false; TC5_STOP }   // they have landed
         unsigned char* vrow = sV + (j % STAGES) * KV_BYTES + r * 128;
 #pragma unroll
         for (int c = 0; c < 8; ++c) {
@@ -435,6 +471,7 @@ paged_prefill_tc5_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
       __syncwarp();
       if (lane == 0) bar_arrive(&p_ready[j & 1]);
     }
+#undef TC5_STOP
     if (ok && n_tiles > 1 && !bar_wait(&pv_done[n_tiles & 1], ((n_tiles - 2) >> 1) & 1)) { atomicExch(error, 16); ok = false; }
     if (ok && n_tiles > 0 && !bar_wait(&pv_done[(n_tiles - 1) & 1], ((n_tiles - 1) >> 1) & 1)) { atomicExch(error, 16); ok = false; }
   }
@@ -475,7 +512,11 @@ paged_prefill_tc5_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
       const float mm = fmaxf(m, m1);
       const float f0 = m == -INFINITY ? 0.f : exp2f(m - mm), f1 = (m1 == -INFINITY || l1 == 0.f) ? 0.f : exp2f(m1 - mm);
       // with the keys cut into chunks the sum stays unnormalised (relative to the reference mm): the merge kernel divides
-      const float inv = n_chunks > 1 ? 1.f : 1.f / (l * f0 + l1 * f1);
+      float inv = n_chunks > 1 ? 1.f : 1.f / (l * f0 + l1 * f1);
+      if (sinks && n_chunks == 1) {      // the sink joins the denominator only: with the larger of the two as the reference
+        const float sk = sinks[h] * 1.4426950408889634f, ms = fmaxf(mm, sk), keep = exp2f(mm - ms);
+        inv = keep / fmaf(l * f0 + l1 * f1, keep, exp2f(sk - ms));
+      }
       const float g0 = f0 * inv, g1 = f1 * inv;
       asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
       __nv_bfloat16* dst = out + (size_t)(r_begin + tile * BM + r) * out_ld + h * HD;
@@ -566,26 +607,29 @@ CBIS_EXPORT int cbis_paged_prefill_tc5(const void* q, int q_ld, int total_rows, 
                                        const int* seg_start, void* out, int out_ld, int seg0, int n_seg,
                                        int max_seg_rows, int n_head, int n_kv_head, int hd, int ps, float scale,
                                        int window, int n_chunks, int chunk_keys, float* partial, const int* positions,
-                                       int row0, int n_rows, int* error, void* stream) {
+                                       int row0, int n_rows, int* error, void* stream, const float* sinks,
+                                       const float* slopes, const float* rates, int v_heads) {
   if (n_seg <= 0 || max_seg_rows <= 0) return CBIS_OK;
   if (n_chunks < 1 || (n_chunks > 1 && (chunk_keys <= 0 || chunk_keys % tc5::BN || !partial || !positions || n_rows <= 0 ||
                                         ((uintptr_t)partial & 15))))
     return CBIS_ERR_BAD_SIZE;
-  if ((hd != 128 && hd != 64) || ps < 8 || ps > 128 || (ps & (ps - 1)) || n_head <= 0 || n_kv_head <= 0 || n_head % n_kv_head)
+  if ((hd != 128 && hd != 64) || ps < 8 || ps > 128 || (ps & (ps - 1)) || n_head <= 0 || n_kv_head <= 0 ||
+      (v_heads != 1 && (v_heads != n_kv_head || n_head % v_heads)) || (n_head / v_heads) % n_kv_head || !slopes != !rates)
     return CBIS_ERR_BAD_SIZE;
   if (q_ld % 8 || out_ld % 8 || ((uintptr_t)q & 15) || ((uintptr_t)kc & 15) || ((uintptr_t)vc & 15) ||
       ((uintptr_t)out & 15) || error == nullptr)
     return CBIS_ERR_ALIGNMENT;
   CUtensorMap map_q, map_k, map_v;
-  int st = tc5::make_map(&map_q, q, total_rows, n_head * hd, q_ld, tc5::BM);
+  int st = tc5::make_map(&map_q, q, total_rows, n_head / v_heads * hd, q_ld, tc5::BM);
   if (st != CBIS_OK) return st;
   const long long cache_rows = (long long)num_pages * n_kv_head * ps;
   st = tc5::make_map(&map_k, kc, cache_rows, hd, hd, ps < tc5::BN ? ps : tc5::BN);
   if (st != CBIS_OK) return st;
   st = tc5::make_map(&map_v, vc, cache_rows, hd, hd, ps < tc5::BN ? ps : tc5::BN);
   if (st != CBIS_OK) return st;
-  const size_t smem = tc5::smem_bytes(hd);
-  auto kern = hd == 128 ? tc5::paged_prefill_tc5_kernel<128> : tc5::paged_prefill_tc5_kernel<64>;
+  const size_t smem = tc5::smem_bytes(hd) + (rates ? tc5::TABLE * sizeof(float) : 0);
+  auto kern = hd == 128 ? (rates ? tc5::paged_prefill_tc5_kernel<128, true> : tc5::paged_prefill_tc5_kernel<128, false>)
+                        : (rates ? tc5::paged_prefill_tc5_kernel<64, true> : tc5::paged_prefill_tc5_kernel<64, false>);
   cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
   if (e != cudaSuccess) return (int)e;
   e = cudaFuncSetAttribute(kern, cudaFuncAttributePreferredSharedMemoryCarveout, (int)cudaSharedmemCarveoutMaxShared);
@@ -593,11 +637,11 @@ CBIS_EXPORT int cbis_paged_prefill_tc5(const void* q, int q_ld, int total_rows, 
   dim3 grid(2u * (unsigned)((max_seg_rows + tc5::BM - 1) / tc5::BM) * n_head * n_seg * n_chunks);
   e = launch_pdl(kern, grid, dim3(tc5::THREADS), smem, (cudaStream_t)stream, map_q, map_k, map_v, block_table, max_blocks,
                  cu_rows, seg_start, (__nv_bfloat16*)out, out_ld, seg0, n_seg, n_head, n_kv_head, ps,
-                 scale * 1.4426950408889634f, window, n_chunks, chunk_keys, partial, row0, error);
+                 scale * 1.4426950408889634f, window, n_chunks, chunk_keys, partial, row0, error, sinks, slopes, rates, v_heads);
   if (e == cudaSuccess && n_chunks > 1)
     e = launch_pdl(prefill_merge_kernel<__nv_bfloat16, true>, dim3(n_rows), dim3(128), 0, (cudaStream_t)stream,
                    (const float*)partial, positions, (const int*)nullptr, (__nv_bfloat16*)out, out_ld, row0, n_head, hd, window,
-                   n_chunks, chunk_keys, (const float*)nullptr);
+                   n_chunks, chunk_keys, sinks);
   return (int)e;
 }
 
@@ -606,7 +650,7 @@ CBIS_EXPORT int cbis_paged_prefill_tc5(const void* q, int q_ld, int total_rows, 
 // memory) and what the device's SMs have; negative: a CUDA error.  (The occupancy calls of the runtime answer for
 // whole clusters and count an SM pair once; the profiler's counters show two blocks per SM at work.)
 CBIS_EXPORT int cbis_paged_prefill_tc5_blocks_per_sm() {
-  auto kern = tc5::paged_prefill_tc5_kernel<128>;
+  auto kern = tc5::paged_prefill_tc5_kernel<128, false>;
   cudaFuncAttributes fa;
   cudaError_t e = cudaFuncGetAttributes(&fa, kern);
   if (e != cudaSuccess) return -(int)e;

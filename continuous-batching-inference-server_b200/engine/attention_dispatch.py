@@ -18,8 +18,8 @@ positions, counted from position 0: the query sees its own block's keys up to p)
 A mixer may also name (attributes, all optional): ``v_head_dim`` (values of another width than the keys; with one
 cached array for keys and values the values are the first entries of its rows), ``slopes`` (a distance bias per
 head; with ``rates`` it grows with the logarithm of the distance), ``sinks`` (a number per head in the softmax's
-denominator), ``q_temp`` (a query temperature by position) and ``v_heads`` (n_kv_head: every query head attends to the
-values of every key/value head; the heads of the kernels, of ``out`` and of the numbers per head are then these pairs).
+denominator), ``q_temp`` (a query temperature by position) and ``talk`` (the softmax weights are mixed across heads; the
+mixer may then hand over a gate on the result, element by element).
 ``run_attention`` returns how many columns a head's result takes in ``out``.
 """
 from __future__ import annotations
@@ -52,11 +52,14 @@ def _general_chunks(ctx, n_head, rows, hd):
 
 
 def _extended(ctx, mixer, qkv, cache, view, out, k_pages, v_pages, k_off, v_off, vd, slopes, sinks, q_temp,
-              rates, v_heads) -> int:
-    """Attention with values of their own width, a distance bias, a sink or a query temperature.  bfloat16 with
-    widths that are multiples of 8: the decoding rows go to the split-KV decode kernel's lane-group form (up to 256
-    wide; it stores the current token's key and value itself), the longer segments, after the cache-write kernel, to
-    the tiled tensor-core kernel (up to 128 wide, pages of a power of two).  32-bit, other sizes: the cache-write
+              rates, v_heads=1, done=0) -> int:
+    """Attention with values of their own width, a distance bias, a sink or a query temperature; with ``v_heads`` =
+    n_kv_head every query head over the values of every key/value head (the heads of ``out`` and of the numbers per head
+    are then these pairs); rows before ``done`` (0 or the decoding rows) have been taken care of.  bfloat16 with
+    widths that are multiples of 8: the decoding rows go to the split-KV decode kernel (up to 256 wide; it stores
+    the current token's key and value itself), the longer segments, after the cache-write kernel, to the TMA + tcgen05
+    kernel (head sizes 64 and 128, no temperature, no linear bias) or the tiled tensor-core kernel (up to 128 wide, pages of
+    a power of two).  32-bit, other sizes: the cache-write
     kernel and the general kernel."""
     T, nd, hd, ps = ctx.n_rows, ctx.n_decode, mixer.head_dim, cache.page_size
     extra = dict(v_head_dim=vd, slopes=slopes, sinks=sinks, q_temp=q_temp, rates=rates, v_heads=v_heads)
@@ -64,9 +67,9 @@ def _extended(ctx, mixer, qkv, cache, view, out, k_pages, v_pages, k_off, v_off,
     o = out[:, :n_head * vd]
     by8 = (qkv.dtype == torch.bfloat16 and hd % 8 == 0 and vd % 8 == 0 and qkv.stride(0) % 8 == 0 and k_off % 8 == 0
            and v_off % 8 == 0 and qkv.data_ptr() % 16 == 0 and o.stride(0) % 8 == 0 and o.data_ptr() % 16 == 0)
-    fast_decode = by8 and nd > 0 and max(hd, vd) <= 256
+    fast_decode = by8 and nd > 0 and max(hd, vd) <= 256 and not done
     tiled = by8 and T > nd and max(hd, vd) <= 128 and ps & (ps - 1) == 0 and ops.USE_TILED_EXTENDED
-    first = nd if fast_decode else 0        # rows from here on have their keys and values stored by the cache-write kernel
+    first = nd if fast_decode else done     # rows from here on have their keys and values stored by the cache-write kernel
     if fast_decode:
         nsplit = ops.decode_splits(nd, n_head, ctx.ctx_limit)
         scratch = counters = None
@@ -80,6 +83,14 @@ def _extended(ctx, mixer, qkv, cache, view, out, k_pages, v_pages, k_off, v_off,
     r = slice(first, T)
     if mixer.own_kv:
         ops.kv_write(qkv[r], k_off, v_off, k_pages, v_pages, view.slot_mapping[r], mixer.n_kv_head, hd, ps, v_head_dim=vd)
+    tc5 = (tiled and first == nd and hd == vd and hd in (64, 128) and 8 <= ps <= 128 and ops.USE_TCGEN05 and q_temp is None
+           and (slopes is None) == (rates is None) and k_pages is not v_pages and o.data_ptr() % 16 == 0)
+    if tc5:          # TMA + tcgen05: takes a sink, a bias that grows with the logarithm of the distance, all value heads
+        chunks, partial = _key_chunks(ctx, n_head, nd, T, hd, row_tile=128, blocks_per_tile=2, blocks_per_sm=2, min_chunk=8192)
+        ops.paged_prefill_tc5(qkv, k_pages, v_pages, view.block_table, ctx.cu_rows, ctx.seg_start, o, nd, ctx.n_segments - nd,
+                              ctx.max_seg_rows, n_head, mixer.n_kv_head, hd, ps, mixer.scale, mixer.window, chunks, partial,
+                              ctx.positions, nd, T - nd, sinks=sinks, slopes=slopes, rates=rates, v_heads=v_heads)
+        return vd
     if tiled:        # q and out keep their full row numbering, the kernel finds its rows through cu_rows
         chunks, partial = _key_chunks(ctx, n_head, first, T, vd)
         ops.paged_prefill_bf16(qkv, k_pages, v_pages, view.block_table, ctx.cu_rows, ctx.seg_start, o, first,
@@ -93,9 +104,40 @@ def _extended(ctx, mixer, qkv, cache, view, out, k_pages, v_pages, k_off, v_off,
     return vd
 
 
-def run_attention(ctx, mixer, qkv, cache, view, out) -> int:
+def _mixed(ctx, mixer, qkv, cache, view, out, gate) -> int:
+    """Attention whose softmax weights are mixed across heads (``talk``): decoding rows in bfloat16 by the pair of
+    kernels that mixes the weights themselves; the other rows run every query head over the values of every key/value
+    head (``v_heads`` of ``_extended``) and the results are mixed, the two sums exchanged."""
+    T, nd, vd, H, G = ctx.n_rows, ctx.n_decode, mixer.v_head_dim, mixer.n_head, mixer.n_kv_head
+    hd, ps = mixer.head_dim, cache.page_size
+    k_pages, v_pages = cache.arrays["k"], cache.arrays["v"]
+    k_off, v_off = (mixer.d_q, mixer.d_q + mixer.d_kv) if mixer.own_kv else (-1, -1)
+    cap = -(-ctx.ctx_limit // 16) * 16
+    first = 0
+    if (nd > 0 and ops.decode_mix_takes(qkv.dtype, nd, H, hd, vd, cap) and qkv.stride(0) % 8 == 0 and qkv.data_ptr() % 16 == 0
+            and all(o < 0 or o % 8 == 0 for o in (k_off, v_off))):
+        blocks = ops.decode_mix_blocks(H, G)
+        nsplit = ops.decode_splits(nd, blocks, ctx.ctx_limit)
+        scratch, counters = ctx.decode_scratch(ops.decode_mix_scratch_floats(nd, H, vd, cap, nsplit), nd * blocks)
+        ops.decode_mix_bf16(qkv[:nd], k_off, v_off, k_pages, v_pages, view.block_table, ctx.row_seq, ctx.positions,
+                            view.slot_mapping, mixer.talk, mixer.sinks, None if gate is None else gate[:nd], out[:nd], scratch,
+                            counters, cap, H, G, hd, vd, ps, mixer.scale, mixer.window, nsplit)
+        first = nd
+    if first >= T:
+        return vd
+    every = torch.empty((T, H * G * vd), dtype=out.dtype, device=out.device)
+    _extended(ctx, mixer, qkv, cache, view, every, k_pages, v_pages, mixer.d_q, mixer.d_q + mixer.d_kv, vd, None,
+              mixer.sinks_every, None, None, G, done=first)
+    r = slice(first, T)
+    ops.mix_heads(every[r], mixer.talk, H, G, vd, out[r], None if gate is None else gate[r])
+    return vd
+
+
+def run_attention(ctx, mixer, qkv, cache, view, out, gate=None) -> int:
     nd = ctx.n_decode
     T = ctx.n_rows
+    if getattr(mixer, "talk", None) is not None:
+        return _mixed(ctx, mixer, qkv, cache, view, out, gate)
     hd, ps = mixer.head_dim, cache.page_size
     # the pages that stand for keys and for values: "k" and "v", or what the mixer names (a mixer whose keys and
     # values are both one cached array names it twice)
@@ -105,10 +147,8 @@ def run_attention(ctx, mixer, qkv, cache, view, out) -> int:
     v_off = k_off if v_name == k_name else k_off + mixer.d_kv      # one array for both: one column block for both
     vd = int(getattr(mixer, "v_head_dim", 0) or hd)
     slopes, sinks, q_temp, rates = (getattr(mixer, a, None) for a in ("slopes", "sinks", "q_temp", "rates"))
-    v_heads = int(getattr(mixer, "v_heads", 1))
-    if vd != hd or slopes is not None or sinks is not None or q_temp is not None or v_heads > 1:
-        return _extended(ctx, mixer, qkv, cache, view, out, k_pages, v_pages, k_off, v_off, vd, slopes, sinks, q_temp, rates,
-                         v_heads)
+    if vd != hd or slopes is not None or sinks is not None or q_temp is not None:
+        return _extended(ctx, mixer, qkv, cache, view, out, k_pages, v_pages, k_off, v_off, vd, slopes, sinks, q_temp, rates)
     _plain(ctx, mixer, qkv, cache, view, out, nd, T, hd, ps, k_pages, v_pages, k_off, v_off)
     return hd
 

@@ -86,9 +86,10 @@ class StepContext:
     def layer_state(self, li: int):
         return self.pool.state.get(li)
 
-    def attention(self, mixer, qkv, cache, view, out):
-        """Stores this step's keys/values of ``mixer`` (if it keeps its own) and attends over the pages."""
-        return run_attention(self, mixer, qkv, cache, view, out)
+    def attention(self, mixer, qkv, cache, view, out, gate=None):
+        """Stores this step's keys/values of ``mixer`` (if it keeps its own) and attends over the pages.  ``gate``: for a
+        mixer whose weights are mixed across heads, an element-wise gate on the result."""
+        return run_attention(self, mixer, qkv, cache, view, out, gate)
 
     def decode_scratch(self, n_floats: int, n_counters: int):
         """(float scratch, zeroed int32 counters) for kernels that split work and merge it in the last block."""

@@ -494,6 +494,13 @@ def kv_write(qkv, k_off, v_off, k_cache, v_cache, slot_mapping, n_kv_head, head_
     _check(st, "kv_write", f"T={T} kv_heads={n_kv_head} head_dim={head_dim} page={page_size}")
 
 
+def _need_columns(q, out, n_head, v_heads, head_dim, v_head_dim):
+    """The launch's heads have their queries in q and their results in out."""
+    if q.shape[1] < n_head // v_heads * head_dim or out.shape[1] < n_head * v_head_dim:
+        raise KernelError(f"attention: {n_head} heads ({v_heads} value heads a query head) of {head_dim} and {v_head_dim} do not fit "
+                          f"rows of {q.shape[1]} and {out.shape[1]} columns")
+
+
 def generic_key_chunks(rows: int, n_head: int, max_context: int, head_dim: int):
     """(n_chunks, chunk_keys) for the general attention kernel (a warp per row and head): no cut (1, 0) when rows and
     heads alone give 16 warps to each of the 148 SMs, or the head size is no multiple of 4; else chunks of a power
@@ -531,6 +538,7 @@ def paged_attention_generic(q, k_cache, v_cache, block_table, row_seq, positions
     if n_head % (n_kv_head * v_heads):
         raise KernelError(f"attention: n_head={n_head} is not a multiple of n_kv_head={n_kv_head}")
     assert q.stride(1) == 1 and out.stride(1) == 1 and block_table.dtype == torch.int32
+    _need_columns(q, out, n_head, v_heads, head_dim, int(v_head_dim) or head_dim)
     assert block_table.is_contiguous() and row_seq.dtype == torch.int32 and positions.dtype == torch.int32
     n_chunks, chunk_keys = chunks
     vd = int(v_head_dim) or head_dim
@@ -585,6 +593,7 @@ def paged_decode_bf16(qkv, k_off, v_off, k_cache, v_cache, block_table, row_seq,
     for t in (slopes, sinks, rates):
         assert t is None or (t.dtype == torch.float32 and t.numel() == n_head)
     coef, every = q_temp if q_temp else (0.0, 0)
+    _need_columns(qkv, out, n_head, v_heads, head_dim, vd)
     if nsplit > 1:
         assert scratch.dtype == torch.float32 and scratch.numel() >= decode_scratch_floats(rows, n_head, vd, nsplit)
         assert counters.dtype == torch.int32 and counters.numel() >= rows * n_head
@@ -596,6 +605,55 @@ def paged_decode_bf16(qkv, k_off, v_off, k_cache, v_cache, block_table, row_seq,
         c_int(int(v_head_dim)), c_int(v_cache.shape[-1]), _ptr(slopes), _ptr(sinks), c_float(coef), c_int(int(every)),
         _ptr(rates), c_int(v_heads))
     _check(st, "paged_decode_bf16", f"rows={rows} heads={n_head}/{n_kv_head} head_dim={head_dim} splits={nsplit}")
+
+
+USE_DECODE_MIX = __import__("os").environ.get("CBIS_DECODE_MIX", "1") != "0"   # 0: decoding rows whose weights are mixed across heads run every head over every value head and mix the results
+DECODE_MIX_MAX_SCRATCH = 1 << 29      # the most bytes of scores a decode step may take
+
+
+def decode_mix_blocks(n_head: int, n_kv_head: int) -> int:
+    """Blocks per row and split of the second kernel of ``decode_mix_bf16`` (the counters a row needs)."""
+    return int(kernels().cbis_decode_mix_blocks(c_int(n_head), c_int(n_kv_head)))
+
+
+def decode_mix_scratch_floats(rows: int, n_head: int, v_head_dim: int, cap: int, nsplit: int) -> int:
+    fn = kernels().cbis_decode_mix_scratch_floats
+    fn.restype = ctypes.c_longlong
+    return int(fn(c_int(rows), c_int(n_head), c_int(v_head_dim), c_int(cap), c_int(nsplit)))
+
+
+def decode_mix_takes(dtype, rows: int, n_head: int, head_dim: int, v_head_dim: int, cap: int) -> bool:
+    """Whether ``decode_mix_bf16`` takes these sizes."""
+    return (USE_DECODE_MIX and dtype == torch.bfloat16 and head_dim % 8 == 0 and v_head_dim % 8 == 0
+            and max(head_dim, v_head_dim) <= 256 and n_head <= 128 and rows * n_head * cap * 4 <= DECODE_MIX_MAX_SCRATCH)
+
+
+def decode_mix_bf16(qkv, k_off, v_off, k_cache, v_cache, block_table, row_seq, positions, slot_mapping, talk, sinks, gate, out,
+                    scratch, counters, cap, n_head, n_kv_head, head_dim, v_head_dim, page_size, scale, window, nsplit):
+    """Decode attention (one query per row) whose softmax weights are mixed across heads, w'_h = sum_g talk[h, g] w_g,
+    before head h applies them to its own key/value head's values; ``sinks`` (per head, or None) join the denominators
+    unmixed; ``gate`` ``[rows, n_head * v_head_dim]`` (or None): the result times sigmoid(gate).  With ``k_off`` / ``v_off``
+    >= 0 the current token's key / value are taken from ``qkv`` and stored.  ``cap``: a multiple of 16, no less than the
+    longest request; ``scratch``: ``decode_mix_scratch_floats`` floats; ``counters``: rows * ``decode_mix_blocks`` int32,
+    zero before the first launch (every launch leaves them zero)."""
+    _need_cuda(qkv, k_cache, v_cache, block_table, row_seq, positions, slot_mapping, talk, sinks, gate, out, scratch, counters)
+    rows = qkv.shape[0]
+    assert qkv.dtype == torch.bfloat16 == out.dtype == k_cache.dtype and qkv.stride(1) == 1 and out.stride(1) == 1
+    _need_columns(qkv, out, n_head, 1, head_dim, v_head_dim)
+    assert k_cache.shape[1] == n_kv_head == v_cache.shape[1] and k_cache.shape[3] == head_dim and v_cache.shape[3] == v_head_dim
+    assert talk.dtype == torch.float32 and talk.shape == (n_head, n_head) and talk.is_contiguous()
+    assert sinks is None or (sinks.dtype == torch.float32 and sinks.numel() == n_head)
+    assert gate is None or (gate.dtype == torch.bfloat16 and gate.shape == (rows, n_head * v_head_dim) and gate.stride(1) == 1)
+    assert scratch.dtype == torch.float32 and scratch.numel() >= decode_mix_scratch_floats(rows, n_head, v_head_dim, cap, nsplit)
+    assert nsplit == 1 or (counters.dtype == torch.int32 and counters.numel() >= rows * decode_mix_blocks(n_head, n_kv_head))
+    assert block_table.is_contiguous() and block_table.dtype == torch.int32
+    st = kernels().cbis_decode_mix_bf16(
+        _ptr(qkv), c_int(qkv.stride(0)), c_int(k_off), c_int(v_off), _ptr(k_cache), _ptr(v_cache), _ptr(block_table),
+        c_int(block_table.shape[1]), _ptr(row_seq), _ptr(positions), _ptr(slot_mapping), _ptr(talk), _ptr(sinks), _ptr(gate),
+        c_int(gate.stride(0) if gate is not None else 0), _ptr(out), c_int(out.stride(0)), _ptr(scratch), _ptr(counters),
+        c_int(cap), c_int(rows), c_int(n_head), c_int(n_kv_head), c_int(head_dim), c_int(v_head_dim), c_int(page_size),
+        c_float(scale), c_int(window), c_int(nsplit), _stream())
+    _check(st, "decode_mix_bf16", f"rows={rows} heads={n_head}/{n_kv_head} widths={head_dim}/{v_head_dim} splits={nsplit}", launches=2)
 
 
 def paged_prefill_bf16(q, k_cache, v_cache, block_table, cu_rows, seg_start, out, seg0, n_seg, max_seg_rows,
@@ -621,6 +679,7 @@ def paged_prefill_bf16(q, k_cache, v_cache, block_table, cu_rows, seg_start, out
     assert q.dtype == torch.bfloat16 and k_cache.dtype == torch.bfloat16 and out.dtype == torch.bfloat16
     assert q.stride(1) == 1 and out.stride(1) == 1 and block_table.is_contiguous()
     v_row = v_cache.shape[-1]
+    _need_columns(q, out, n_head, v_heads, head_dim, vd)
     for t in (slopes, sinks, rates):
         assert t is None or (t.dtype == torch.float32 and t.numel() == n_head and t.is_cuda)
     coef, every = q_temp if q_temp else (0.0, 0)
@@ -686,11 +745,12 @@ def paged_prefill_f32(q, k_cache, v_cache, block_table, cu_rows, seg_start, out,
 
 def paged_prefill_tc5(q, k_cache, v_cache, block_table, cu_rows, seg_start, out, seg0, n_seg, max_seg_rows,
                       n_head, n_kv_head, head_dim, page_size, scale, window=0, chunks=(1, 0), partial=None,
-                      positions=None, row0=0, n_rows=0):
+                      positions=None, row0=0, n_rows=0, sinks=None, slopes=None, rates=None, v_heads=1):
     """The same attention as ``paged_prefill_bf16`` on the tcgen05 tensor cores (TMA operands, S and the output in
     tensor memory).  Head size 64 or 128, page sizes 8..128 (powers of two); ``q`` and ``out`` in full row numbering.
     ``chunks``, ``partial``, ``positions``, ``row0``, ``n_rows`` as for ``paged_prefill_bf16`` (chunks from
-    ``prefill_key_chunks`` with two blocks per 128-row tile, two per SM and chunks of at least 8,192 keys)."""
+    ``prefill_key_chunks`` with two blocks per 128-row tile, two per SM and chunks of at least 8,192 keys);
+    ``sinks``, ``slopes`` with ``rates``, ``v_heads`` as in ``paged_attention_generic``."""
     _need_cuda(q, k_cache, v_cache, block_table, cu_rows, seg_start, out, partial, positions)
     if head_dim not in (64, 128):
         raise KernelError(f"tcgen05 prefill attention: head_dim={head_dim} is neither 64 nor 128")
@@ -698,6 +758,9 @@ def paged_prefill_tc5(q, k_cache, v_cache, block_table, cu_rows, seg_start, out,
         raise KernelError(f"tcgen05 prefill attention: page_size={page_size} is not a power of two in 8..128")
     assert q.dtype == torch.bfloat16 and k_cache.dtype == torch.bfloat16 and out.dtype == torch.bfloat16
     assert q.stride(1) == 1 and out.stride(1) == 1 and block_table.is_contiguous() and k_cache.is_contiguous()
+    _need_columns(q, out, n_head, v_heads, head_dim, head_dim)
+    for t in (sinks, slopes, rates):
+        assert t is None or (t.dtype == torch.float32 and t.numel() == n_head and t.is_cuda)
     n_chunks, chunk_keys = chunks
     if n_chunks > 1:
         assert partial.dtype == torch.float32 and partial.numel() >= n_rows * n_head * n_chunks * (head_dim + 4)
@@ -707,7 +770,8 @@ def paged_prefill_tc5(q, k_cache, v_cache, block_table, cu_rows, seg_start, out,
         _ptr(block_table), c_int(block_table.shape[1]), _ptr(cu_rows), _ptr(seg_start), _ptr(out),
         c_int(out.stride(0)), c_int(seg0), c_int(n_seg), c_int(max_seg_rows), c_int(n_head), c_int(n_kv_head),
         c_int(head_dim), c_int(page_size), c_float(scale), c_int(window), c_int(n_chunks), c_int(chunk_keys),
-        _ptr(partial), _ptr(positions), c_int(row0), c_int(n_rows), _ptr(tcgen05_error_flag(q.device)), _stream())
+        _ptr(partial), _ptr(positions), c_int(row0), c_int(n_rows), _ptr(tcgen05_error_flag(q.device)), _stream(), _ptr(sinks),
+        _ptr(slopes), _ptr(rates), c_int(v_heads))
     _check(st, "paged_prefill_tc5", f"segments={n_seg} heads={n_head}/{n_kv_head} page={page_size} chunks={n_chunks}x{chunk_keys}")
 
 

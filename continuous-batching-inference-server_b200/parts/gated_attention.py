@@ -32,8 +32,9 @@ class GatedAttention(Mixer):
     * ``sinks``: a learned number per head whose exponential joins the softmax's denominator (no key, no value).
     * ``talk``: the softmax weights are mixed across heads by a learned matrix T ``[n_head, n_head]`` before they meet the
       values: w'_h = sum_g T[h, g] w_g, head h applies w'_h to its own key/value head's values; sinks are not mixed.
-      The attention kernels give every query head's sum over the values of EVERY key/value head (``v_heads``), and
-      one more kernel takes the sum over g (and the element gate): the order of the two sums is exchanged.
+      Decoding rows in bfloat16 mix the weights themselves; elsewhere the attention kernels give every query head's sum
+      over the values of EVERY key/value head, and one more kernel takes the sum over g (and the element gate): the order
+      of the two sums is exchanged.
     * ``own_kv`` False: the layer has no keys and values of its own (projections, their norm): it reads the pages of the
       layer its cache source names, with its own queries and everything else.
 
@@ -67,12 +68,11 @@ class GatedAttention(Mixer):
         self.has_sinks, self.has_talk = bool(sinks), bool(talk)
         if self.has_talk and self.n_head > ops.MIX_HEADS_MAX_HEADS:
             raise ValueError(f"n_head={n_head} is above {ops.MIX_HEADS_MAX_HEADS}, the most heads whose weights are mixed")
-        # how many value heads the attention kernels run every query head over
-        self.v_heads = self.n_kv_head if self.has_talk else 1
         self.d_q, self.d_kv, self.d_v = self.n_head * self.head_dim, self.n_kv_head * self.head_dim, self.n_kv_head * self.v_head_dim
         self.names = tuple(names) + NAMES[len(tuple(names)):]
         self.w_in = self.b_in = self.w_out = self.b_out = None
         self.q_norm_w = self.k_norm_w = self.slopes = self.rates = self.sinks = self.talk = None
+        self.sinks_every = None      # with talk: a number per (query head, value head), for kernels that run every such pair
 
     def cache_need(self):
         if not self.own_kv:
@@ -125,19 +125,18 @@ class GatedAttention(Mixer):
         if self.qk_norm:
             self.q_norm_w = self._vector(tensors[n[0] + ".norm"], device)
             self.k_norm_w = self._vector(tensors[n[1] + ".norm"], device) if self.own_kv else None
-
-        def per_launch_head(t):      # a number per head, for every value head the kernels run it over
-            return t.repeat_interleave(self.v_heads).contiguous()
         if self.slope_power:
-            self.slopes = per_launch_head(torch.tensor([2.0 ** (-self.slope_power * (h + 1) / self.n_head) for h in range(self.n_head)],
-                                                       dtype=torch.float64).to(torch.float32).to(device))
+            self.slopes = torch.tensor([2.0 ** (-self.slope_power * (h + 1) / self.n_head) for h in range(self.n_head)],
+                                       dtype=torch.float64).to(torch.float32).to(device)
         if self.log_bias:
-            self.slopes = per_launch_head(self._vector(tensors[n[5]], device))
-            self.rates = per_launch_head(self._vector(tensors[n[6]], device))
+            self.slopes = self._vector(tensors[n[5]], device)
+            self.rates = self._vector(tensors[n[6]], device)
         if self.has_sinks:
-            self.sinks = per_launch_head(self._vector(tensors[n[7]], device))
+            self.sinks = self._vector(tensors[n[7]], device)
         if self.has_talk:
             self.talk = self._vector(tensors[n[8]], device)
+            if self.has_sinks:
+                self.sinks_every = self.sinks.repeat_interleave(self.n_kv_head).contiguous()
 
     def streamed_weights(self):
         return [self.w_in, self.w_out]
@@ -151,14 +150,11 @@ class GatedAttention(Mixer):
         if self.qk_norm:
             ops.qk_head_norm(proj, 0, self.n_head, self.d_q, self.n_kv_head if self.own_kv else 0, self.head_dim,
                              self.q_norm_w, self.k_norm_w, self.eps)
-        out = torch.empty((T, HV * self.v_heads), dtype=h.dtype, device=h.device)
-        ctx.attention(self, proj, cache, ctx.groups[cache.group], out)     # stores k and v (if its own), then attends
+        out = torch.empty((T, HV), dtype=h.dtype, device=h.device)
         gate = proj[:, gate0:gate0 + HV] if self.gate == "element" else None
-        if self.has_talk:
-            mixed = torch.empty((T, HV), dtype=h.dtype, device=h.device)
-            ops.mix_heads(out, self.talk, self.n_head, self.v_heads, self.v_head_dim, mixed, gate)
-            out = mixed
-        elif gate is not None:
+        inside = gate if self.has_talk else None      # the kernels that mix the heads apply the gate too
+        ctx.attention(self, proj, cache, ctx.groups[cache.group], out, gate=inside)     # stores k and v (if its own), then attends
+        if gate is not None and inside is None:
             ops.gate_mul(gate, out, "sigmoid", out)
         if self.gate == "head":
             ops.head_gate_mul(out, proj[:, gate0:gate0 + self.n_head], self.n_head, out)
