@@ -81,7 +81,8 @@ mix_heads_kernel(const TT* o, int o_ld, const float* __restrict__ talk, const TT
 #pragma unroll
       for (int k = 0; k < V; ++k) acc[u][k] = 0.f;
     const int n = min(HG, (a + 1) * group - h0);
-    for (int g = 0; g < H; ++g) {
+#pragma unroll 8
+    for (int g = 0; g < H; ++g) {      // eight loads in flight
       const Pack<TT, V> p = *reinterpret_cast<const Pack<TT, V>*>(src + (size_t)g * G * vd);
 #pragma unroll
       for (int u = 0; u < HG; ++u) {
