@@ -181,29 +181,35 @@ mix_values_kernel(const __nv_bfloat16* qkv, int ld, int v_off, __nv_bfloat16* vc
       *reinterpret_cast<uint4*>(vc + (((size_t)(slot / ps) * n_kv_head + a) * ps + slot % ps) * vd + tid * 8) =
           *reinterpret_cast<const uint4*>(qkv + (size_t)row * ld + v_off + a * vd + tid * 8);
   }
-  for (int h = tid; h < n_head; h += blockDim.x) {
-    const float2* st = stats + ((size_t)row * n_head + h) * nsplit;
-    const float sink = sinks ? sinks[h] : -INFINITY;
-    float m = sink, l = sinks ? 1.f : 0.f;
-    for (int s = 0; s < nsplit; ++s) {
-      const float2 v = st[s];
-      if (v.x > -INFINITY) {
-        const float mm = fmaxf(m, v.x);
-        l = l * expf(m - mm) + v.y * expf(v.x - mm);
-        m = mm;
-      }
+  __syncthreads();                            // the current token's value is stored
+  constexpr int GW = 32 / LPK, UB = LPK < (NQ > 4 ? 4 : 8) ? LPK : (NQ > 4 ? 4 : 8);
+  const int sub = lane % LPK, grp = lane / LPK;
+  const bool active = sub * 8 < vd;
+  uint4 vn[UB];
+  auto fetch = [&](int base, int it0) {       // this lane's pieces of UB of the warp's 32 / GW value rows
+#pragma unroll
+    for (int i = 0; i < UB; ++i) {
+      const int j = base + warp * 32 + (it0 + i) * GW + grp;
+      vn[i] = make_uint4(0, 0, 0, 0);
+      if (active && j < ke) vn[i] = ldcg16(vc + (((size_t)bt[j / ps] * n_kv_head + a) * ps + j % ps) * vd + sub * 8);
     }
-    top[h] = m;
-    inv[h] = 1.f / l;
+  };
+  fetch(ks, 0);                               // on their way while the heads' sums and the first weights are computed
+  for (int h = warp; h < n_head; h += DEC_WARPS) {      // a warp a head, a lane a split (32 at most)
+    const float2 v = lane < nsplit ? stats[((size_t)row * n_head + h) * nsplit + lane] : make_float2(-INFINITY, 0.f);
+    const float sink = sinks ? sinks[h] : -INFINITY;
+    const float m = fmaxf(warp_max(v.x), sink);
+    const float l = warp_sum(v.x > -INFINITY ? v.y * expf(v.x - m) : 0.f) + (sinks ? expf(sink - m) : 0.f);
+    if (lane == 0) {
+      top[h] = m;
+      inv[h] = 1.f / l;
+    }
   }
   __syncthreads();
   for (int i = tid; i < NQ * n_head; i += blockDim.x) {
     const int u = i / n_head, gh = i % n_head;
     tw[i] = u < nq ? talk[(size_t)(h0 + u) * n_head + gh] * inv[gh] : 0.f;
   }
-  constexpr int GW = 32 / LPK, UB = LPK < (NQ > 4 ? 4 : 8) ? LPK : (NQ > 4 ? 4 : 8);
-  const int sub = lane % LPK, grp = lane / LPK;
-  const bool active = sub * 8 < vd;
   float acc[NQ][8];
 #pragma unroll
   for (int u = 0; u < NQ; ++u)
@@ -211,23 +217,14 @@ mix_values_kernel(const __nv_bfloat16* qkv, int ld, int v_off, __nv_bfloat16* vc
     for (int i = 0; i < 8; ++i) acc[u][i] = 0.f;
   for (int base = ks; base < ke; base += MIX_KEYS) {
     __syncthreads();                          // tw is there; wmix of the keys before has been read
-    uint4 vn[UB];
-    auto fetch = [&](int it0, uint4* v) {     // this lane's pieces of UB of the warp's 32 / GW value rows
-#pragma unroll
-      for (int i = 0; i < UB; ++i) {
-        const int j = base + warp * 32 + (it0 + i) * GW + grp;
-        v[i] = make_uint4(0, 0, 0, 0);
-        if (active && j < ke) v[i] = ldcg16(vc + (((size_t)bt[j / ps] * n_kv_head + a) * ps + j % ps) * vd + sub * 8);
-      }
-    };
-    fetch(0, vn);
     {
       float w[NQ];
 #pragma unroll
       for (int u = 0; u < NQ; ++u) w[u] = 0.f;
       if (base + tid < ke) {
         const float* s = scores + (size_t)row * n_head * cap + base + tid;
-        for (int gh = 0; gh < n_head; ++gh) {
+#pragma unroll 8
+        for (int gh = 0; gh < n_head; ++gh) {      // eight scores in flight
           const float e = expf(s[(size_t)gh * cap] - top[gh]);
 #pragma unroll
           for (int u = 0; u < NQ; ++u) w[u] = fmaf(tw[u * n_head + gh], e, w[u]);
@@ -242,7 +239,8 @@ mix_values_kernel(const __nv_bfloat16* qkv, int ld, int v_off, __nv_bfloat16* vc
       uint4 v[UB];
 #pragma unroll
       for (int i = 0; i < UB; ++i) v[i] = vn[i];
-      if (it0 + UB < LPK) fetch(it0 + UB, vn);
+      if (it0 + UB < LPK) fetch(base, it0 + UB);
+      else if (base + MIX_KEYS < ke) fetch(base + MIX_KEYS, 0);
 #pragma unroll
       for (int i = 0; i < UB; ++i) {
         float f[8];
@@ -292,10 +290,21 @@ mix_values_kernel(const __nv_bfloat16* qkv, int ld, int v_off, __nv_bfloat16* vc
   __syncthreads();
   if (!is_last) return;
   __threadfence();
-  for (int i = tid; i < nq * vd; i += blockDim.x) {
-    float v = 0.f;
-    for (int s = 0; s < nsplit; ++s) v += __ldcg(mine + ((size_t)(i / vd) * nsplit + s) * vd + i % vd);
-    store(i, v);
+  for (int i = tid * 4; i < nq * vd; i += blockDim.x * 4) {
+    const float4* src = reinterpret_cast<const float4*>(mine + (size_t)(i / vd) * nsplit * vd + i % vd);
+    float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 8
+    for (int s = 0; s < nsplit; ++s) {         // eight loads in flight, added in their order
+      const float4 p = __ldcg(src + (size_t)s * (vd / 4));
+      v.x += p.x;
+      v.y += p.y;
+      v.z += p.z;
+      v.w += p.w;
+    }
+    store(i, v.x);
+    store(i + 1, v.y);
+    store(i + 2, v.z);
+    store(i + 3, v.w);
   }
   if (tid == 0) *counter = 0;
 }
@@ -315,7 +324,7 @@ CBIS_EXPORT int cbis_decode_mix_blocks(int n_head, int n_kv_head) {
 // Floats of scratch for `rows` rows: every head's scores of up to `cap` keys (a multiple of 16), the splits' maxima and
 // sums, and their partial results.
 CBIS_EXPORT long long cbis_decode_mix_scratch_floats(int rows, int n_head, int vd, int cap, int nsplit) {
-  return (long long)rows * n_head * cap + (long long)rows * n_head * nsplit * (2 + (nsplit > 1 ? vd : 0));
+  return (long long)rows * n_head * cap + (long long)rows * n_head * nsplit * (2 + (nsplit > 1 ? vd : 0)) + 2;
 }
 
 // qkv: this step's projections [rows, ld], queries at column 0; k_off / v_off >= 0: the current token's key / value are
@@ -338,7 +347,7 @@ CBIS_EXPORT int cbis_decode_mix_bf16(const void* qkv, int ld, int k_off, int v_o
   cudaStream_t st = (cudaStream_t)stream;
   float* scores = scratch;
   float2* stats = reinterpret_cast<float2*>(scores + (size_t)rows * n_head * cap);
-  float* part = reinterpret_cast<float*>(stats + (size_t)rows * n_head * nsplit);
+  float* part = reinterpret_cast<float*>(stats + (((size_t)rows * n_head * nsplit + 1) & ~(size_t)1));      // 16-byte aligned
   typedef __nv_bfloat16 bf;
   cudaError_t e = cudaErrorInvalidValue;
 #define CBIS_SC(NC)                                                                                                   \
