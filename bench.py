@@ -1089,7 +1089,7 @@ def fororax_kernels(torch, ops, pk):
             r = torch.empty(B, nh * hd, dtype=bf, device="cuda")
             if mixing:
                 blocks = ops.decode_mix_blocks(nh, nkv)
-                ns = ops.decode_splits(B, blocks, ctx_len)
+                ns = ops.decode_mix_splits(B, nh, nkv, ctx_len)
                 scratch = torch.empty(ops.decode_mix_scratch_floats(B, nh, hd, ctx_len, ns), device="cuda")
                 counters = torch.zeros(B * blocks, dtype=torch.int32, device="cuda")
                 return lambda: ops.decode_mix_bf16(qkv, nh * hd, (nh + nkv) * hd, k, v, btB, row_seq, posB, slot_map, talk, sinks,

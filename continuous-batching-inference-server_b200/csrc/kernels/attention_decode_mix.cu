@@ -146,7 +146,7 @@ mix_scores_kernel(const __nv_bfloat16* qkv, int ld, int k_off, __nv_bfloat16* kc
 // grid (rows, n_kv_head * pieces of NQ of the heads that share a value head, nsplit).  LPK lanes a value row (8 entries
 // each).  Dynamic shared memory: 2 H floats, NQ * H, NQ * MIX_KEYS, DEC_WARPS * NQ * vd.
 template <int LPK, int NQ>
-__global__ void __launch_bounds__(DEC_WARPS * 32)
+__global__ void __launch_bounds__(DEC_WARPS * 32, NQ <= 4 ? 4 : 2)      // four blocks per SM, what the splits are sized for
 mix_values_kernel(const __nv_bfloat16* qkv, int ld, int v_off, __nv_bfloat16* vc, const int* block_table, int max_blocks,
                   const int* row_seq, const int* positions, const int* slot_mapping, const float* scores, int cap,
                   const float2* stats, const float* __restrict__ talk, const float* __restrict__ sinks,

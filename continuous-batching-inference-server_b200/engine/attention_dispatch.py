@@ -117,7 +117,7 @@ def _mixed(ctx, mixer, qkv, cache, view, out, gate) -> int:
     if (nd > 0 and ops.decode_mix_takes(qkv.dtype, nd, H, hd, vd, cap) and qkv.stride(0) % 8 == 0 and qkv.data_ptr() % 16 == 0
             and all(o < 0 or o % 8 == 0 for o in (k_off, v_off))):
         blocks = ops.decode_mix_blocks(H, G)
-        nsplit = ops.decode_splits(nd, blocks, ctx.ctx_limit)
+        nsplit = ops.decode_mix_splits(nd, H, G, ctx.ctx_limit)
         scratch, counters = ctx.decode_scratch(ops.decode_mix_scratch_floats(nd, H, vd, cap, nsplit), nd * blocks)
         ops.decode_mix_bf16(qkv[:nd], k_off, v_off, k_pages, v_pages, view.block_table, ctx.row_seq, ctx.positions,
                             view.slot_mapping, mixer.talk, mixer.sinks, None if gate is None else gate[:nd], out[:nd], scratch,

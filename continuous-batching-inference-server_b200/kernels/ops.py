@@ -616,6 +616,12 @@ def decode_mix_blocks(n_head: int, n_kv_head: int) -> int:
     return int(kernels().cbis_decode_mix_blocks(c_int(n_head), c_int(n_kv_head)))
 
 
+def decode_mix_splits(rows: int, n_head: int, n_kv_head: int, max_context: int) -> int:
+    """How many ways ``decode_mix_bf16`` splits a request's keys: one round of blocks, four of them on an SM, two where
+    more than four query heads share a key/value head (a block then holds eight heads' sums)."""
+    return decode_splits(rows, decode_mix_blocks(n_head, n_kv_head) * (1 if n_head // n_kv_head <= 4 else 2), max_context)
+
+
 def decode_mix_scratch_floats(rows: int, n_head: int, v_head_dim: int, cap: int, nsplit: int) -> int:
     fn = kernels().cbis_decode_mix_scratch_floats
     fn.restype = ctypes.c_longlong
