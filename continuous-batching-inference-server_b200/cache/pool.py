@@ -50,11 +50,13 @@ class CacheGroup:
 
 def _need_with_readers(model, li: int, need: CacheNeed) -> CacheNeed:
     """A layer's pages stay as long as the layer itself OR a layer that reads its cache can reach them: the
-    window that decides when pages go back is the widest of theirs (0, no window, is the widest of all)."""
-    windows = [need.window] + [int(getattr(other.mixer, "window", 0)) for other in model.layers
-                               if other.spec.cache_source == li]
+    window that decides when pages go back is the widest of theirs (0, no window, is the widest of all), and the first
+    tokens that stay are the most that one of them goes on seeing."""
+    readers = [other.mixer for other in model.layers if other.spec.cache_source == li]
+    windows = [need.window] + [int(getattr(m, "window", 0)) for m in readers]
     widest = 0 if any(w <= 0 for w in windows) else max(windows)
-    return need if widest == need.window else replace(need, window=widest)
+    keep = max([need.keep_first] + [int(getattr(m, "keep_first", 0)) for m in readers]) if widest else 0
+    return need if (widest, keep) == (need.window, need.keep_first) else replace(need, window=widest, keep_first=keep)
 
 
 def cache_groups_of(model, page_size: int) -> List[CacheGroup]:
@@ -107,7 +109,7 @@ class CachePool:
                     arrays[a.name] = g.storage[at:at + n].view(g.num_pages, a.heads, page_size, a.width)
                     at += size
                 self.layer_cache[li] = LayerCache(gi, arrays, page_size, g.need.window)
-            specs.append(host().GroupSpec(page_size, g.num_pages, g.need.window))
+            specs.append(host().GroupSpec(page_size, g.num_pages, g.need.window, g.need.keep_first))
         if not specs:  # a model without any cache still needs request slots and lengths: pages that are counted only
             specs.append(host().GroupSpec(page_size, int(num_pages), 0))
         for li, layer in enumerate(model.layers):

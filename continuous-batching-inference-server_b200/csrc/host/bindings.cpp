@@ -13,17 +13,19 @@ PYBIND11_MODULE(_cbis_host, m) {
   m.doc() = "Host runtime: paged cache manager with groups and state slots, continuous-batching scheduler";
 
   py::class_<GroupSpec>(m, "GroupSpec")
-      .def(py::init([](int page_size, int num_pages, int window) {
+      .def(py::init([](int page_size, int num_pages, int window, int keep_first) {
              GroupSpec g;
              g.page_size = page_size;
              g.num_pages = num_pages;
              g.window = window;
+             g.keep_first = keep_first;
              return g;
            }),
-           py::arg("page_size"), py::arg("num_pages"), py::arg("window") = 0)
+           py::arg("page_size"), py::arg("num_pages"), py::arg("window") = 0, py::arg("keep_first") = 0)
       .def_readwrite("page_size", &GroupSpec::page_size)
       .def_readwrite("num_pages", &GroupSpec::num_pages)
-      .def_readwrite("window", &GroupSpec::window);
+      .def_readwrite("window", &GroupSpec::window)
+      .def_readwrite("keep_first", &GroupSpec::keep_first);
 
   py::class_<CacheManager>(m, "CacheManager")
       .def(py::init<std::vector<GroupSpec>, int>(), py::arg("groups"), py::arg("max_requests"))
@@ -32,6 +34,7 @@ PYBIND11_MODULE(_cbis_host, m) {
       .def("page_size", &CacheManager::page_size)
       .def("num_pages", &CacheManager::num_pages)
       .def("window", &CacheManager::window)
+      .def("keep_first", &CacheManager::keep_first)
       .def("free_pages", &CacheManager::free_pages)
       .def("free_slots", &CacheManager::free_slots)
       .def("admit", &CacheManager::admit)

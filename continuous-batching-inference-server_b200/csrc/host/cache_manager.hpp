@@ -19,6 +19,7 @@ struct GroupSpec {
   int page_size = 16;
   int num_pages = 0;
   int window = 0;  // 0: every earlier key stays reachable; w > 0: the query at p reads keys p-w+1..p
+  int keep_first = 0;  // with a window: the first keys of a sequence that stay reachable behind it
 };
 
 class CacheManager {
@@ -28,7 +29,7 @@ class CacheManager {
     if (groups_.empty()) throw std::invalid_argument("CacheManager: at least one cache group is needed");
     for (size_t g = 0; g < groups_.size(); ++g) {
       const GroupSpec& s = groups_[g];
-      if (s.page_size <= 0 || s.num_pages < 0 || s.window < 0)
+      if (s.page_size <= 0 || s.num_pages < 0 || s.window < 0 || s.keep_first < 0)
         throw std::invalid_argument("CacheManager: bad sizes in group " + std::to_string(g));
       std::vector<int> fl;
       fl.reserve(s.num_pages);
@@ -47,6 +48,7 @@ class CacheManager {
   int page_size(int g) const { return groups_.at(g).page_size; }
   int num_pages(int g) const { return groups_.at(g).num_pages; }
   int window(int g) const { return groups_.at(g).window; }
+  int keep_first(int g) const { return groups_.at(g).keep_first; }
   int free_pages(int g) const { return (int)free_.at(g).size(); }
   int free_slots() const { return (int)free_slots_.size(); }
   int largest_page() const {
@@ -112,13 +114,14 @@ class CacheManager {
   }
   // Whether a request that grows to `n` tokens, written in portions of at most `chunk`, can be
   // held when every other page is free.  A windowed group holds at most the window, the
-  // portion being written and one page of rounding at a time.
+  // portion being written, one page of rounding and the pages of the first keys it keeps at a time.
   bool fits_at_all(int n, int chunk) const {
     for (int g = 0; g < num_groups(); ++g) {
       const GroupSpec& s = groups_[g];
       long live_tokens = n;
       if (s.window > 0) {
-        const long bound = (long)s.window + chunk + s.page_size;
+        const long kept = (long)(s.keep_first + s.page_size - 1) / s.page_size * s.page_size;
+        const long bound = (long)s.window + chunk + s.page_size + kept;
         if (bound < live_tokens) live_tokens = bound;
       }
       if (pages_for(g, (int)live_tokens) > s.num_pages) return false;
@@ -144,7 +147,8 @@ class CacheManager {
     return true;
   }
 
-  // Gives back the pages of windowed groups that no query at position >= length can reach.
+  // Gives back the pages of windowed groups that no query at position >= length can reach (pages with one of the first
+  // keys that stay reachable are never given back).
   // Call it after the step that wrote up to `length` has been put together.
   int release_out_of_window(int slot) {
     Slot& sl = mut(slot);
@@ -153,7 +157,7 @@ class CacheManager {
       const GroupSpec& s = groups_[g];
       if (s.window <= 0) continue;
       const int first_needed = sl.length - s.window + 1;  // first key of the next query
-      for (size_t lp = 0; lp < sl.tables[g].size(); ++lp) {
+      for (size_t lp = (size_t)((s.keep_first + s.page_size - 1) / s.page_size); lp < sl.tables[g].size(); ++lp) {
         if ((long)(lp + 1) * s.page_size > first_needed) break;
         int& p = sl.tables[g][lp];
         if (p >= 0) {

@@ -19,6 +19,9 @@
 // tokens' values), a distance bias (slope[h] * (p - j) taken off the score), a query temperature by position and a
 // sink in the denominator.  The bias may grow with the logarithm of the distance instead (rates), and with v_heads > 1
 // every query head attends to the values of every key/value head (head_place in common.cuh).
+//
+// Both forms take a cap on the scaled scores, cap * tanh(s / cap), and first keys that stay visible behind a window (keep):
+// the keys are then walked, and split, as ONE run, the kept ones first.
 #include "attention_decode_tc.cuh"
 #include <math.h>
 
@@ -37,7 +40,7 @@ paged_decode_bf16_kernel(const __nv_bfloat16* qkv, int ld, int k_off, int v_off,
                          unsigned int* counters, int n_head, int n_kv_head, int hd, int ps, float scale,
                          int window, int nsplit, int hdv, int v_row, const float* __restrict__ slopes,
                          const float* __restrict__ sinks, float temp_coef, int temp_every, const float* __restrict__ rates,
-                         int v_heads) {
+                         int v_heads, float cap, int keep) {
   constexpr int G = 32 / LPK;             // key groups per warp
   constexpr int NW = DEC_WARPS * G;       // key workers per block
   __shared__ float sm_m[DEC_WARPS], sm_l[DEC_WARPS];
@@ -57,10 +60,13 @@ paged_decode_bf16_kernel(const __nv_bfloat16* qkv, int ld, int k_off, int v_off,
   const int hk = hp.key, hv = hp.value;
   const int pos = positions[row];
   const int kend = pos + 1;
-  const int kstart = first_seen(pos, window);
-  const int per = (((kend - kstart) + nsplit - 1) / nsplit + 31) & ~31;
-  const int ks = kstart + split * per;
-  const int ke = min(kend, ks + per);
+  const int kstart = first_seen(pos, window), n_kept = kept_end(pos, window, keep);
+  // ks, ke and the loops count along the keys this row sees: number i is key i of the kept ones, then kstart + i - n_kept
+  const int n_keys = n_kept + kend - kstart;
+  const int per = ((n_keys + nsplit - 1) / nsplit + 31) & ~31;
+  const int ks = split * per;
+  const int ke = min(n_keys, ks + per);
+  auto key_at = [&](int i) { return i < n_kept ? i : kstart + i - n_kept; };
   const int sub = lane % LPK, group = lane / LPK;
   const bool active = sub * 8 < hd, active_v = sub * 8 < hdv;
   const int* bt = block_table + (size_t)seq * max_blocks;
@@ -87,10 +93,10 @@ paged_decode_bf16_kernel(const __nv_bfloat16* qkv, int ld, int k_off, int v_off,
   auto fetch = [&](int base, uint4* kk, uint4* vv) {
 #pragma unroll
     for (int u = 0; u < DEC_U; ++u) {
-      const int j = base + u * NW + wkr;
+      const int i = base + u * NW + wkr, j = key_at(i);
       kk[u] = make_uint4(0, 0, 0, 0);
       vv[u] = make_uint4(0, 0, 0, 0);
-      if (j < ke && (active || active_v)) {
+      if (i < ke && (active || active_v)) {
         if (fused && j == pos) {
           if (active) kk[u] = *reinterpret_cast<const uint4*>(qkv + (size_t)row * ld + k_off + hk * hd + sub * 8);
           if (active_v) vv[u] = *reinterpret_cast<const uint4*>(qkv + (size_t)row * ld + v_off + hv * hdv + sub * 8);
@@ -132,7 +138,8 @@ paged_decode_bf16_kernel(const __nv_bfloat16* qkv, int ld, int k_off, int v_off,
       for (int i = 0; i < 8; ++i) d = fmaf(q[i], kf[i], d);
 #pragma unroll
       for (int o = LPK / 2; o > 0; o >>= 1) d += __shfl_xor_sync(0xffffffffu, d, o);
-      s[u] = valid[u] ? (slope != 0.f ? d - distance_bias(slope, rate, (float)(pos - (base + u * NW + wkr))) : d) : -INFINITY;
+      d = capped_score(d, cap);
+      s[u] = valid[u] ? (slope != 0.f ? d - distance_bias(slope, rate, (float)(pos - key_at(base + u * NW + wkr))) : d) : -INFINITY;
     }
     float m_new = m;
 #pragma unroll
@@ -243,19 +250,19 @@ paged_decode_bf16_kernel(const __nv_bfloat16* qkv, int ld, int k_off, int v_off,
 // The fast form for head sizes 64 and 128 and pages of a multiple of 16 keys: decode_tc_item of
 // attention_decode_tc.cuh, one block of four warps per (row, head, split).
 // ---------------------------------------------------------------------------------------------
-template <int HD, bool BIAS>
+template <int HD, bool BIAS, bool EXT>
 __global__ void __launch_bounds__(DEC_WARPS * 32, 4)   // 128 registers: four blocks per SM
 paged_decode_tc_kernel(const __nv_bfloat16* qkv, int ld, int k_off, int v_off, __nv_bfloat16* kc, __nv_bfloat16* vc,
                        const int* block_table, int max_blocks, const int* row_seq, const int* positions,
                        const int* slot_mapping, __nv_bfloat16* __restrict__ out, int out_ld, float* part,
                        unsigned int* counters, int n_head, int n_kv_head, int ps, float scale, int window,
                        int nsplit, const float* __restrict__ sinks, const float* __restrict__ slopes,
-                       const float* __restrict__ rates) {
+                       const float* __restrict__ rates, float cap, int keep) {
   __shared__ DecodeTcShared<HD> sm;
   pdl_trigger();
-  decode_tc_item<HD, true, (HD <= 64 ? 2 : 1), BIAS>(qkv, ld, k_off, v_off, kc, vc, block_table, max_blocks, row_seq, positions, slot_mapping, out,
+  decode_tc_item<HD, true, (HD <= 64 ? 2 : 1), BIAS, EXT>(qkv, ld, k_off, v_off, kc, vc, block_table, max_blocks, row_seq, positions, slot_mapping, out,
                            out_ld, part, counters, n_head, n_kv_head, ps, scale, window, nsplit, blockIdx.x, blockIdx.y,
-                           blockIdx.z, threadIdx.x, sm, 0, sinks, slopes, rates);
+                           blockIdx.z, threadIdx.x, sm, 0, sinks, slopes, rates, cap, keep);
 }
 
 // After a decode step whose next tokens were chosen on the device: the chosen token becomes the
@@ -310,13 +317,16 @@ CBIS_EXPORT int cbis_paged_decode_bf16(const void* qkv, int ld, int k_off, int v
                                        float* part, unsigned int* counters, int rows, int n_head, int n_kv_head,
                                        int hd, int ps, float scale, int window, int nsplit, void* stream, int hdv,
                                        int v_row, const float* slopes, const float* sinks, float temp_coef,
-                                       int temp_every, const float* rates, int v_heads) {
+                                       int temp_every, const float* rates, int v_heads, float cap, int keep) {
   if (rows <= 0) return CBIS_OK;
   // hdv (0: the keys' width, values in pages of their own): the values' width.  With values of another width or in
   // the keys' rows, a linear bias or a temperature the lane-group form runs whatever the head size; a sink (it joins
-  // the denominator where the parts are merged) and a bias that grows with the logarithm are taken by both forms
+  // the denominator where the parts are merged), a bias that grows with the logarithm, and a cap or kept first keys (not
+  // together with such a bias) are taken by both forms
   if (hdv <= 0) hdv = hd, v_row = hd;
   const bool extended = hdv != hd || v_row != hd || (slopes && !rates) || temp_every > 0 || v_heads > 1;
+  const bool ext = cap > 0.f || (keep > 0 && window != 0);
+  if (keep < 0) return CBIS_ERR_BAD_SIZE;
   if (v_heads != 1 && (v_heads != n_kv_head || n_head % v_heads)) return CBIS_ERR_BAD_SIZE;
   if (hdv > 256 || hdv % 8 || v_row < hdv || v_row % 8) return CBIS_ERR_BAD_SIZE;
   if (hd <= 0 || hd > 256 || hd % 8 || ps <= 0 || n_head <= 0 || n_kv_head <= 0 || (n_head / v_heads) % n_kv_head || nsplit < 1 || nsplit > 32)
@@ -329,19 +339,21 @@ CBIS_EXPORT int cbis_paged_decode_bf16(const void* qkv, int ld, int k_off, int v
   dim3 grid(rows, n_head, nsplit);
   const int chunks = (hd > hdv ? hd : hdv) / 8;
   cudaError_t e;
-  if ((hd == 64 || hd == 128) && ps % 16 == 0 && !extended) {
-    auto kern = hd == 128 ? (slopes ? paged_decode_tc_kernel<128, true> : paged_decode_tc_kernel<128, false>)
-                          : (slopes ? paged_decode_tc_kernel<64, true> : paged_decode_tc_kernel<64, false>);
+  if ((hd == 64 || hd == 128) && ps % 16 == 0 && !extended && !(ext && slopes)) {
+    auto kern = hd == 128 ? (slopes ? paged_decode_tc_kernel<128, true, false>
+                                    : (ext ? paged_decode_tc_kernel<128, false, true> : paged_decode_tc_kernel<128, false, false>))
+                          : (slopes ? paged_decode_tc_kernel<64, true, false>
+                                    : (ext ? paged_decode_tc_kernel<64, false, true> : paged_decode_tc_kernel<64, false, false>));
     return (int)launch_pdl(kern, grid, dim3(DEC_WARPS * 32), 0, st, (const __nv_bfloat16*)qkv, ld, k_off,
                      v_off, (__nv_bfloat16*)kc, (__nv_bfloat16*)vc, block_table, max_blocks, row_seq, positions,
                      slot_mapping, (__nv_bfloat16*)out, out_ld, part, counters, n_head, n_kv_head, ps, scale, window,
-                     nsplit, sinks, slopes, rates);
+                     nsplit, sinks, slopes, rates, cap, keep);
   }
 #define CBIS_DEC(LPK)                                                                                             \
   e = launch_pdl(paged_decode_bf16_kernel<LPK>, grid, dim3(DEC_WARPS * 32), 0, st, (const __nv_bfloat16*)qkv, ld, \
                  k_off, v_off, (__nv_bfloat16*)kc, (__nv_bfloat16*)vc, block_table, max_blocks, row_seq, positions, \
                  slot_mapping, (__nv_bfloat16*)out, out_ld, part, counters, n_head, n_kv_head, hd, ps, scale, window, \
-                 nsplit, hdv, v_row, slopes, sinks, temp_coef, temp_every, rates, v_heads)
+                 nsplit, hdv, v_row, slopes, sinks, temp_coef, temp_every, rates, v_heads, cap, keep)
   if (chunks <= 2) CBIS_DEC(2);
   else if (chunks <= 4) CBIS_DEC(4);
   else if (chunks <= 8) CBIS_DEC(8);

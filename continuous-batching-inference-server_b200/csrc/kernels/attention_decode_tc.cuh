@@ -77,7 +77,11 @@ struct DecodeTcShared {
 // hardware barrier the group meets at.  STANDALONE: the group is a block launched for this alone, which waits for
 // the kernels ahead (programmatic dependent launch) after it has fetched what they do not write.  The group's
 // threads must have met (group_sync) between two calls, since the calls share `sm`.
-template <int HD, bool STANDALONE, int TPW = 1, bool BIAS = false>
+//
+// EXT: a cap on the scaled scores, and first keys that stay visible behind a window (keep).  The tiles are then numbered
+// along what the row sees, the nk tiles that hold kept keys first: tiles, ks, ke and kend are such numbers, `real_tile`
+// says which tile of the sequence one is.
+template <int HD, bool STANDALONE, int TPW = 1, bool BIAS = false, bool EXT = false>
 __device__ __forceinline__ void decode_tc_item(const __nv_bfloat16* qkv, int ld, int k_off, int v_off, __nv_bfloat16* kc,
                                                __nv_bfloat16* vc, const int* block_table, int max_blocks,
                                                const int* row_seq, const int* positions, const int* slot_mapping,
@@ -86,7 +90,8 @@ __device__ __forceinline__ void decode_tc_item(const __nv_bfloat16* qkv, int ld,
                                                int row, int h, int split, int tid, DecodeTcShared<HD>& sm, int bar,
                                                const float* __restrict__ sinks = nullptr,
                                                const float* __restrict__ slopes = nullptr,
-                                               const float* __restrict__ rates = nullptr) {
+                                               const float* __restrict__ rates = nullptr, float cap = 0.f,
+                                               int keep = 0) {
   constexpr int NC = HD / 32;        // 16-byte loads per key for the score fragments (4 lanes x 16 B = 32 dims each)
   constexpr int LPK = HD / 8;        // lanes per key in the coalesced V loads
   constexpr int KPL = 32 / LPK;      // keys per warp-wide V load
@@ -109,11 +114,16 @@ __device__ __forceinline__ void decode_tc_item(const __nv_bfloat16* qkv, int ld,
   }
   const int hk = h / (n_head / n_kv_head);
   const int pos = positions[row];
-  const int kend = pos + 1;
   const int kstart = first_seen(pos, window);
+  const int kept = EXT ? kept_end(pos, window, keep) : 0;
   const int first_tile = kstart >> 4;
-  const int per = (((kend - (first_tile << 4)) + nsplit - 1) / nsplit + 31) & ~31;   // keys per split, whole tiles
-  const int ks = (first_tile << 4) + split * per;
+  const int nk = EXT ? min((kept + 15) >> 4, first_tile) : 0;
+  const int skipped = EXT ? first_tile - nk : 0;             // tiles between the kept ones and the first in the window
+  const int first_numbered = EXT ? 0 : first_tile;
+  auto real_tile = [&](int tile) { return EXT && tile >= nk ? tile + skipped : tile; };
+  const int kend = pos + 1 - (skipped << 4), pos_n = pos - (skipped << 4);
+  const int per = (((kend - (first_numbered << 4)) + nsplit - 1) / nsplit + 31) & ~31;   // keys per split, whole tiles
+  const int ks = (first_numbered << 4) + split * per;
   const int ke = min(kend, ks + per);
   const int* bt = block_table + (size_t)seq * max_blocks;
   const int g = lane >> 2, t = lane & 3;
@@ -128,8 +138,8 @@ __device__ __forceinline__ void decode_tc_item(const __nv_bfloat16* qkv, int ld,
   auto load_keys = [&](int tile) {
 #pragma unroll
     for (int u = 0; u < TPW; ++u) {
-      const int j0 = (tile + u) << 4;
-      if (j0 < ke) {
+      const int j0 = real_tile(tile + u) << 4;
+      if (((tile + u) << 4) < ke) {
         const int pi = ps_shift >= 0 ? (j0 >> ps_shift) : j0 / ps;      // a shift where the page size is a power of two
         base[u] = (((size_t)bt[pi] * n_kv_head + hk) * ps + (j0 - pi * ps)) * HD;   // 16 keys from here are one run
 #pragma unroll
@@ -150,7 +160,7 @@ __device__ __forceinline__ void decode_tc_item(const __nv_bfloat16* qkv, int ld,
   };
   int tile = (ks >> 4) + warp * TPW;
   // not the tiles that hold the current token: its key and value are stored below, after the wait
-  const bool preloaded = (tile << 4) < ke && ((pos >> 4) < tile || (pos >> 4) >= tile + TPW);
+  const bool preloaded = (tile << 4) < ke && ((pos_n >> 4) < tile || (pos_n >> 4) >= tile + TPW);
   if (preloaded) {
     load_keys(tile);
     load_values(tile);
@@ -159,7 +169,7 @@ __device__ __forceinline__ void decode_tc_item(const __nv_bfloat16* qkv, int ld,
 
   // The current token's key and value go into their page first; the loop below then reads them
   // like any other key.  (Blocks of query heads that share this key/value head store the same values.)
-  if (k_off >= 0 && pos >= ks && pos < ke) {
+  if (k_off >= 0 && pos_n >= ks && pos_n < ke) {
     const int slot = slot_mapping[row];
     if (slot >= 0 && tid < 2 * LPK) {
       const int which = tid / LPK, sub = tid % LPK;
@@ -199,7 +209,7 @@ __device__ __forceinline__ void decode_tc_item(const __nv_bfloat16* qkv, int ld,
     float s4[TPW][4], mx = -INFINITY;
 #pragma unroll
     for (int u = 0; u < TPW; ++u) {
-      const int j0 = (tile + u) << 4;
+      const int j0 = (tile + u) << 4, at = real_tile(tile + u) << 4;
       float sc[2][4];
 #pragma unroll
       for (int nt = 0; nt < 2; ++nt) sc[nt][0] = sc[nt][1] = sc[nt][2] = sc[nt][3] = 0.f;
@@ -214,8 +224,9 @@ __device__ __forceinline__ void decode_tc_item(const __nv_bfloat16* qkv, int ld,
       }
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
-        const int j = j0 + (e >> 1) * 8 + 2 * t + (e & 1);
-        s4[u][e] = (g == 0 && j >= kstart && j < ke) ? sc[e >> 1][e & 1] * scale : -INFINITY;
+        const int o = (e >> 1) * 8 + 2 * t + (e & 1), j = at + o;
+        s4[u][e] = (g == 0 && (j >= kstart || j < kept) && j0 + o < ke) ? sc[e >> 1][e & 1] * scale : -INFINITY;
+        if (EXT && s4[u][e] > -INFINITY) s4[u][e] = capped_score(s4[u][e], cap);
         if (BIAS && g == 0) s4[u][e] -= distance_bias(slope, rate, (float)max(pos - j, 0));
         mx = fmaxf(mx, s4[u][e]);
       }

@@ -11,7 +11,9 @@
 //   * a distance bias: slope[h] * (p - j), or slope[h] * ln(1 + rate[h] * (p - j)), is taken off the scaled score of the
 //     key at j for the query at p;
 //   * a query temperature: the score of the query at p is also multiplied by 1 + coef * ln(floor((p + 1) / every) + 1);
-//   * a sink: exp(sink[h]) counts once in the softmax's denominator and has no value.
+//   * a sink: exp(sink[h]) counts once in the softmax's denominator and has no value;
+//   * a cap: the scaled score becomes cap * tanh(score / cap) (before a bias is taken off).
+// With `keep` the first keys of a sequence stay visible behind the window (kept_end in common.cuh).
 // With v_heads > 1 every query head attends to the values of every key/value head (head_place in common.cuh).
 #include "attention_merge.cuh"
 
@@ -82,7 +84,7 @@ __global__ void paged_attention_generic_kernel(
     const int* positions, TT* __restrict__ out, int out_ld, int n_rows, int n_head, int n_kv_head,
     int hd, int ps, float scale, int window, int n_chunks, int chunk_keys, float* partial,
     int hd_v, int v_row, const float* __restrict__ slopes, const float* __restrict__ sinks, float temp_coef,
-    int temp_every, const float* __restrict__ rates, int v_heads) {
+    int temp_every, const float* __restrict__ rates, int v_heads, float cap, int keep) {
   pdl_trigger();
   pdl_wait();
   const int lane = threadIdx.x & 31;
@@ -107,8 +109,15 @@ __global__ void paged_attention_generic_kernel(
   if (n_chunks > 1) {   // this warp's share of the keys: chunks by absolute index, merged by a second kernel
     kstart = max(kstart, chunk * chunk_keys);
     kend = min(kend, (chunk + 1) * chunk_keys);
-    if (kstart >= kend) return;
   }
+  // the keys are walked as one run: first those kept before the window (kfirst on, n_kept of them), then kstart .. kend - 1
+  const int kfirst = n_chunks > 1 ? chunk * chunk_keys : 0;
+  int n_kept = kept_end(pos, window, keep);
+  if (n_chunks > 1) n_kept = min(n_kept, (chunk + 1) * chunk_keys);
+  n_kept = max(n_kept - kfirst, 0);
+  const int n_keys = n_kept + max(kend - kstart, 0);
+  if (n_chunks > 1 && n_keys <= 0) return;
+  auto key_at = [&](int i) { return i < n_kept ? kfirst + i : kstart + i - n_kept; };
 
   float qv[NPER], acc[NPER];
 #pragma unroll
@@ -119,15 +128,15 @@ __global__ void paged_attention_generic_kernel(
   }
   float m = -INFINITY, l = 0.f;
 
-  for (int j0 = kstart; j0 < kend; j0 += G) {
+  for (int i0 = 0; i0 < n_keys; i0 += G) {
     float s[G];
     const TT* vptr[G];
 #pragma unroll
     for (int u = 0; u < G; ++u) {
-      const int j = j0 + u;
+      const int j = key_at(i0 + u);
       float part = 0.f;
       vptr[u] = nullptr;
-      if (j < kend) {
+      if (i0 + u < n_keys) {
         const int page = bt[j / ps];
         const size_t token = ((size_t)page * n_kv_head + hp.key) * ps + (j % ps);
         const TT* kp = kc + token * hd;
@@ -142,7 +151,12 @@ __global__ void paged_attention_generic_kernel(
     }
 #pragma unroll
     for (int u = 0; u < G; ++u)
-      s[u] = (j0 + u < kend) ? fmaf(warp_sum(s[u]), scale, slope != 0.f ? -distance_bias(slope, rate, (float)(pos - (j0 + u))) : 0.f) : -INFINITY;
+      if (cap > 0.f) {
+        const float a = capped_score(warp_sum(s[u]) * scale, cap);
+        s[u] = i0 + u < n_keys ? (slope != 0.f ? a - distance_bias(slope, rate, (float)(pos - key_at(i0 + u))) : a) : -INFINITY;
+      } else {
+        s[u] = i0 + u < n_keys ? fmaf(warp_sum(s[u]), scale, slope != 0.f ? -distance_bias(slope, rate, (float)(pos - key_at(i0 + u))) : 0.f) : -INFINITY;
+      }
     float m_new = m;
 #pragma unroll
     for (int u = 0; u < G; ++u) m_new = fmaxf(m_new, s[u]);
@@ -151,7 +165,7 @@ __global__ void paged_attention_generic_kernel(
     float psum = 0.f;
 #pragma unroll
     for (int u = 0; u < G; ++u) {
-      p[u] = (j0 + u < kend) ? expf(s[u] - m_new) : 0.f;
+      p[u] = i0 + u < n_keys ? expf(s[u] - m_new) : 0.f;
       psum += p[u];
     }
     l = l * corr + psum;
@@ -231,7 +245,7 @@ static int launch_generic(const void* q, int q_ld, const void* kc, const void* v
                           int n_rows, int n_head, int n_kv_head, int hd, int ps, float scale, int window,
                           int n_chunks, int chunk_keys, float* partial, int hd_v, int v_row, const float* slopes,
                           const float* sinks, float temp_coef, int temp_every, const float* rates, int v_heads,
-                          cudaStream_t st) {
+                          float cap, int keep, cudaStream_t st) {
   const int warps = 4;
   const long long total = (long long)n_rows * n_head * n_chunks;
   const int blocks = (int)((total + warps - 1) / warps);
@@ -240,7 +254,7 @@ static int launch_generic(const void* q, int q_ld, const void* kc, const void* v
   e = launch_pdl(paged_attention_generic_kernel<TT, NPER, (NPER <= 2 ? 16 : (NPER <= 4 ? 8 : (NPER <= 8 ? 4 : 2)))>, dim3(blocks), dim3(warps * 32), 0, st, (const TT*)q, q_ld, \
                  (const TT*)kc, (const TT*)vc, block_table, max_blocks, row_seq, positions, (TT*)out, out_ld, n_rows, \
                  n_head, n_kv_head, hd, ps, scale, window, n_chunks, chunk_keys, partial, hd_v, v_row, slopes, sinks, \
-                 temp_coef, temp_every, rates, v_heads)
+                 temp_coef, temp_every, rates, v_heads, cap, keep)
   const int widest = hd > hd_v ? hd : hd_v;
   if (widest <= 32) CBIS_LAUNCH(1);
   else if (widest <= 64) CBIS_LAUNCH(2);
@@ -250,7 +264,7 @@ static int launch_generic(const void* q, int q_ld, const void* kc, const void* v
 #undef CBIS_LAUNCH
   if (e == cudaSuccess && n_chunks > 1)
     e = launch_pdl(prefill_merge_kernel<TT, false>, dim3(n_rows), dim3(128), 0, st, (const float*)partial, positions, row_seq,
-                   (TT*)out, out_ld, 0, n_head, hd_v, window, n_chunks, chunk_keys, sinks);
+                   (TT*)out, out_ld, 0, n_head, hd_v, window, n_chunks, chunk_keys, sinks, keep);
   return (int)e;
 }
 
@@ -263,10 +277,11 @@ CBIS_EXPORT int cbis_paged_attention_generic(const void* q, int q_ld, const void
                                              int n_kv_head, int hd, int ps, float scale, int window, int dtype,
                                              int n_chunks, int chunk_keys, float* partial, void* stream,
                                              int hd_v, int v_row, const float* slopes, const float* sinks,
-                                             float temp_coef, int temp_every, const float* rates, int v_heads) {
+                                             float temp_coef, int temp_every, const float* rates, int v_heads,
+                                             float cap, int keep) {
   if (n_rows <= 0) return CBIS_OK;
   if (hd_v <= 0) hd_v = hd, v_row = hd;      // values as wide as the keys, in an array of their own
-  if (hd_v > 512 || v_row < hd_v) return CBIS_ERR_BAD_SIZE;
+  if (hd_v > 512 || v_row < hd_v || keep < 0) return CBIS_ERR_BAD_SIZE;
   if (v_heads != 1 && (v_heads != n_kv_head || n_head % v_heads)) return CBIS_ERR_BAD_SIZE;
   if (hd <= 0 || hd > 512 || ps <= 0 || n_head <= 0 || n_kv_head <= 0 || (n_head / v_heads) % n_kv_head) return CBIS_ERR_BAD_SIZE;
   if (n_chunks < 1 || (n_chunks > 1 && (chunk_keys <= 0 || !partial || hd_v % 4 || out_ld % 4 || ((uintptr_t)partial & 15) ||
@@ -276,10 +291,10 @@ CBIS_EXPORT int cbis_paged_attention_generic(const void* q, int q_ld, const void
   if (dtype == CBIS_F32)
     return launch_generic<float>(q, q_ld, kc, vc, block_table, max_blocks, row_seq, positions, out, out_ld, n_rows,
                                  n_head, n_kv_head, hd, ps, scale, window, n_chunks, chunk_keys, partial, hd_v, v_row,
-                                 slopes, sinks, temp_coef, temp_every, rates, v_heads, st);
+                                 slopes, sinks, temp_coef, temp_every, rates, v_heads, cap, keep, st);
   if (dtype == CBIS_BF16)
     return launch_generic<__nv_bfloat16>(q, q_ld, kc, vc, block_table, max_blocks, row_seq, positions, out, out_ld,
                                          n_rows, n_head, n_kv_head, hd, ps, scale, window, n_chunks, chunk_keys, partial, hd_v, v_row,
-                                 slopes, sinks, temp_coef, temp_every, rates, v_heads, st);
+                                 slopes, sinks, temp_coef, temp_every, rates, v_heads, cap, keep, st);
   return CBIS_ERR_BAD_DTYPE;
 }

@@ -16,6 +16,9 @@
 // sink in the denominator, as in the general kernel.  A bias that grows with the logarithm of the distance (rates) is
 // taken from a table of the tile's 127 distances, made once per key tile; with v_heads > 1 every query head attends to the
 // values of every key/value head (head_place in common.cuh).
+//
+// EXT: a cap on the scaled scores, cap * tanh(s / cap), and first keys that stay visible behind a window (keep): the tiles
+// that hold kept keys are walked before those of the window.
 #include "attention_merge.cuh"
 #include <math.h>
 
@@ -62,7 +65,7 @@ __device__ __forceinline__ uint32_t pack_bf16(float lo, float hi) {
 // grid: (row tiles of the longest segment, heads, segments from seg0 on).  cu_rows/seg_start are the
 // step's segment tables: rows cu_rows[s]..cu_rows[s+1] of q/out belong to segment s and start at
 // position seg_start[s].
-template <int HD>
+template <int HD, bool EXT>
 __global__ void __launch_bounds__(PF_WARPS * 32, 3)
 paged_prefill_bf16_kernel(const __nv_bfloat16* q, int q_ld, const __nv_bfloat16* kc, const __nv_bfloat16* vc,
                           const int* block_table, int max_blocks, const int* cu_rows, const int* seg_start,
@@ -70,7 +73,7 @@ paged_prefill_bf16_kernel(const __nv_bfloat16* q, int q_ld, const __nv_bfloat16*
                           float scale_log2e, int window, int n_chunks, int chunk_keys, float* partial, int row0,
                           int hdk, int hdv, int v_row, const float* __restrict__ slopes,
                           const float* __restrict__ sinks, float temp_coef, int temp_every,
-                          const float* __restrict__ rates, int v_heads) {
+                          const float* __restrict__ rates, int v_heads, float cap_log2e, int keep) {
   constexpr int PITCH = HD + 8;  // elements per shared-memory row: 16 bytes of padding keep ldmatrix conflict-free
   constexpr int KS = HD / 16;    // k-steps of Q*K^T
   constexpr int DT = HD / 8;     // 8-wide column tiles of the output
@@ -98,8 +101,22 @@ paged_prefill_bf16_kernel(const __nv_bfloat16* q, int q_ld, const __nv_bfloat16*
   if (n_chunks > 1) {   // this block's share of the keys (chunks by absolute index, whole key tiles)
     kbegin = max(kbegin, chunk * chunk_keys);
     kend = min(kend, (chunk + 1) * chunk_keys);
-    if (kbegin >= kend) return;
+    if (!EXT && kbegin >= kend) return;
   }
+  // the tiles of this block: n_kept tiles from kept_tile on that hold kept keys only, then those of the window
+  const int kept = EXT ? kept_end(pos0, window, keep) : 0;      // of the tile's first row; no later row keeps fewer
+  const int kept_tile = EXT && n_chunks > 1 ? chunk * (chunk_keys / PF_BN) : 0;
+  const int kt_first = kbegin / PF_BN;
+  int n_kept = 0, n_tiles = kbegin < kend ? (kend - 1) / PF_BN - kt_first + 1 : 0;
+  if (EXT) {
+    const int upto = n_chunks > 1 ? min(kept, (chunk + 1) * chunk_keys) : kept;
+    n_kept = max((upto + PF_BN - 1) / PF_BN - kept_tile, 0);
+    if (n_tiles > 0) n_kept = min(n_kept, kt_first - kept_tile);
+    else kend = 0;                                              // no key of the window is in this chunk
+    n_tiles += n_kept;
+    if (n_tiles <= 0) return;
+  }
+  auto tile_at = [&](int i) { return i < n_kept ? kept_tile + i : kt_first + i - n_kept; };
   const int* bt = block_table + (size_t)seg * max_blocks;
 
   // this thread's two rows: g and g + 8 of the warp's 16
@@ -132,7 +149,6 @@ paged_prefill_bf16_kernel(const __nv_bfloat16* q, int q_ld, const __nv_bfloat16*
   for (int d = 0; d < DT; ++d) o[d][0] = o[d][1] = o[d][2] = o[d][3] = 0.f;
   float m0 = -INFINITY, m1 = -INFINITY, l0 = 0.f, l1 = 0.f;
 
-  const int kt_first = kbegin / PF_BN, kt_last = (kend - 1) / PF_BN;
   const int live_from = (kbegin >> ps_shift) << ps_shift;
   auto load_tile = [&](int kt, int stage) {
     __nv_bfloat16* dk = sK + (size_t)stage * PF_BN * PITCH;
@@ -140,7 +156,7 @@ paged_prefill_bf16_kernel(const __nv_bfloat16* q, int q_ld, const __nv_bfloat16*
     for (int idx = threadIdx.x; idx < PF_BN * CHUNKS; idx += PF_WARPS * 32) {
       const int r = idx / CHUNKS, c = idx % CHUNKS;
       const int j = kt * PF_BN + r;
-      const bool valid = j < kend && j >= live_from;   // pages behind the window may have been given back
+      const bool valid = (j < kend && j >= live_from) || (EXT && j < kept);   // pages behind the window may have been given back
       size_t token = 0;
       if (valid) {
         const int page = bt[j >> ps_shift];
@@ -153,11 +169,11 @@ paged_prefill_bf16_kernel(const __nv_bfloat16* q, int q_ld, const __nv_bfloat16*
     cp_async_commit();
   };
 
-  load_tile(kt_first, 0);
-  for (int kt = kt_first; kt <= kt_last; ++kt) {
-    const int stage = (kt - kt_first) & 1;
-    if (kt < kt_last) {
-      load_tile(kt + 1, stage ^ 1);
+  load_tile(tile_at(0), 0);
+  for (int it = 0; it < n_tiles; ++it) {
+    const int kt = tile_at(it), stage = it & 1;
+    if (it + 1 < n_tiles) {
+      load_tile(tile_at(it + 1), stage ^ 1);
       cp_async_wait<1>();
     } else {
       cp_async_wait<0>();
@@ -197,6 +213,10 @@ paged_prefill_bf16_kernel(const __nv_bfloat16* q, int q_ld, const __nv_bfloat16*
       for (int e = 0; e < 2; ++e) {
         const int j = j0 + nt * 8 + 2 * t + e;
         float a = s[nt][e] * sc0, b2 = s[nt][2 + e] * sc1;
+        if constexpr (EXT) {
+          a = capped_score(a, cap_log2e);
+          b2 = capped_score(b2, cap_log2e);
+        }
         if (rates) {
           const int at = PF_BN - 1 - (j - j0);
           a -= s_bias[at + lr0];
@@ -206,8 +226,8 @@ paged_prefill_bf16_kernel(const __nv_bfloat16* q, int q_ld, const __nv_bfloat16*
           b2 = fmaf(-slope2, (float)(p1 - j), b2);
         }
         if (edge) {
-          if (j > p0 || j < lo0) a = -INFINITY;
-          if (j > p1 || j < lo1) b2 = -INFINITY;
+          if (j > p0 || (j < lo0 && !(EXT && j < keep))) a = -INFINITY;
+          if (j > p1 || (j < lo1 && !(EXT && j < keep))) b2 = -INFINITY;
         }
         s[nt][e] = a;
         s[nt][2 + e] = b2;
@@ -305,13 +325,14 @@ CBIS_EXPORT int cbis_paged_prefill_bf16(const void* q, int q_ld, const void* kc,
                                         int window, int n_chunks, int chunk_keys, float* partial, const int* positions,
                                         int row0, int n_rows, void* stream, int hd_v, int v_row,
                                         const float* slopes, const float* sinks, float temp_coef, int temp_every,
-                                        const float* rates, int v_heads) {
+                                        const float* rates, int v_heads, float cap, int keep) {
   if (n_seg <= 0 || max_seg_rows <= 0) return CBIS_OK;
   // hd: the keys' width; hd_v (0: the keys'): the values'; both multiples of 8, the wider of them rounded up to a
   // multiple of 16 picks the tile
   const int hdk = hd;
   if (hd_v <= 0) hd_v = hd, v_row = hd;
-  if (hdk % 8 || hd_v % 8 || v_row < hd_v || v_row % 8) return CBIS_ERR_BAD_SIZE;
+  const bool ext = cap > 0.f || (keep > 0 && window != 0);
+  if (hdk % 8 || hd_v % 8 || v_row < hd_v || v_row % 8 || keep < 0) return CBIS_ERR_BAD_SIZE;
   hd = ((hdk > hd_v ? hdk : hd_v) + 15) / 16 * 16;
   if (n_chunks < 1 || (n_chunks > 1 && (chunk_keys <= 0 || chunk_keys % PF_BN || !partial || !positions || n_rows <= 0 ||
                                         ((uintptr_t)partial & 15) || out_ld % 4 || ((uintptr_t)out & 7))))
@@ -330,7 +351,7 @@ CBIS_EXPORT int cbis_paged_prefill_bf16(const void* q, int q_ld, const void* kc,
   e = cudaErrorInvalidValue;
 #define CBIS_PF(HD_)                                                                                                  \
   if (hd == HD_) {                                                                                                    \
-    auto kern = paged_prefill_bf16_kernel<HD_>;                                                                       \
+    auto kern = ext ? paged_prefill_bf16_kernel<HD_, true> : paged_prefill_bf16_kernel<HD_, false>;                                                                       \
     const size_t smem = (size_t)4 * PF_BN * (HD_ + 8) * sizeof(__nv_bfloat16);                                        \
     if (smem > 48 * 1024) {                                                                                           \
       e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);                         \
@@ -339,12 +360,12 @@ CBIS_EXPORT int cbis_paged_prefill_bf16(const void* q, int q_ld, const void* kc,
     e = launch_pdl(kern, grid, dim3(PF_WARPS * 32), smem, st, (const __nv_bfloat16*)q, q_ld, (const __nv_bfloat16*)kc, \
                    (const __nv_bfloat16*)vc, block_table, max_blocks, cu_rows, seg_start, (__nv_bfloat16*)out, out_ld, seg0, \
                    n_head, n_kv_head, ps_shift, scale_log2e, window, n_chunks, chunk_keys, partial, row0, hdk, hd_v,  \
-                   v_row, slopes, sinks, temp_coef, temp_every, rates, v_heads);                                                      \
+                   v_row, slopes, sinks, temp_coef, temp_every, rates, v_heads, cap * 1.4426950408889634f, keep);                                                      \
   }
   CBIS_PF(16) CBIS_PF(32) CBIS_PF(48) CBIS_PF(64) CBIS_PF(80) CBIS_PF(96) CBIS_PF(112) CBIS_PF(128)
 #undef CBIS_PF
   if (e == cudaSuccess && n_chunks > 1)
     e = launch_pdl(prefill_merge_kernel<__nv_bfloat16, true>, dim3(n_rows), dim3(128), 0, st, (const float*)partial, positions,
-                   (const int*)nullptr, (__nv_bfloat16*)out, out_ld, row0, n_head, hd_v, window, n_chunks, chunk_keys, sinks);
+                   (const int*)nullptr, (__nv_bfloat16*)out, out_ld, row0, n_head, hd_v, window, n_chunks, chunk_keys, sinks, keep);
   return (int)e;
 }

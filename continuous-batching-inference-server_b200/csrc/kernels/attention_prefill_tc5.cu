@@ -30,6 +30,12 @@
 // 64), and a thread reads its row's 64 entries without conflicts.  With v_heads > 1 every query head attends to the values of every key/value
 // head (head_place in common.cuh).
 //
+// EXT: a cap on the scaled scores, cap * tanh(s / cap), and first keys that stay visible behind a window (keep).  The key
+// tiles are numbered along what the row tile sees, the tiles that hold kept keys first, and shared out between the two
+// blocks by that number.  The cap's tanh is a polynomial while the tile's scores are below 3/4 of the cap (normed queries
+// and keys with a cap a few times their largest score always are: six multiply-adds a score, where an exponential and a
+// quotient would triple the load of the special-function units), else it goes through an exponential.
+//
 // Every wait on an mbarrier is bounded; when a limit runs out the block sets *error, stops, frees its
 // tensor memory and returns (its output rows are then invalid, and the host raises).
 #include "attention_merge.cuh"
@@ -163,6 +169,22 @@ __device__ __forceinline__ void tmem_st32(unsigned taddr, const float* v) {
   asm volatile("tcgen05.wait::st.sync.aligned;" ::: "memory");
 }
 
+// x * (polynomial in x^2) = tanh(x) for |x| <= 3/4, from a Chebyshev interpolation of tanh(x) / x in x^2 (sixth
+// coefficient last): relative error below 2e-7.
+constexpr float TANH_POLY_MAX = 0.75f;
+__device__ __forceinline__ float tanh_poly(float x) {
+  const float u = x * x;
+  float r = -0.00472395f;
+  r = fmaf(r, u, 0.01959379f);
+  r = fmaf(r, u, -0.05334982f);
+  r = fmaf(r, u, 0.13325515f);
+  r = fmaf(r, u, -0.33332968f);
+  r = fmaf(r, u, 1.0f);
+  return x * r;
+}
+// 1 - 2 / (e^(2x) + 1): absolute error of a few 1e-7, for any x.
+__device__ __forceinline__ float tanh_exp(float x) { return 1.f - __fdividef(2.f, exp2f(fminf(x * 2.8853900817779268f, 126.f)) + 1.f); }
+
 // The 128 softmax threads (warps 2..5) meet at a barrier of their own.
 __device__ __forceinline__ void softmax_warps_meet() {
   __syncwarp();
@@ -173,14 +195,14 @@ __device__ __forceinline__ void softmax_warps_meet() {
 // blocks of a cluster share a row tile, the first takes the first half of its key tiles and the second the rest,
 // and at the end the second hands its sum, reference and output to the first through distributed shared memory.
 // The row tile with the most keys decides how long the kernel runs, and its chain of tiles is halved this way.
-template <int HD, bool BIAS>
+template <int HD, bool BIAS, bool EXT>
 __global__ void __cluster_dims__(2, 1, 1) __launch_bounds__(THREADS, 2)
 paged_prefill_tc5_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                          const __grid_constant__ CUtensorMap map_v, const int* block_table, int max_blocks,
                          const int* cu_rows, const int* seg_start, __nv_bfloat16* out, int out_ld, int seg0, int n_seg,
                          int n_head, int n_kv_head, int ps, float scale_log2e, int window, int n_chunks, int chunk_keys,
                          float* partial, int row0, int* error, const float* __restrict__ sinks,
-                         const float* __restrict__ slopes, const float* __restrict__ rates, int v_heads) {
+                         const float* __restrict__ slopes, const float* __restrict__ rates, int v_heads, float cap, int keep) {
   constexpr int HALVES = HD / 64, Q_BYTES = HALVES * Q_HALF_BYTES, KV_BYTES = HALVES * KV_HALF_BYTES;
   extern __shared__ __align__(1024) unsigned char base[];   // no byte to spare for rounding the address up: checked below
   unsigned char* sQ = base;                                   // 2 halves of the head dim
@@ -219,11 +241,36 @@ paged_prefill_tc5_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
                         // by absolute index) and leaves an unnormalised partial result for the merge kernel
     kbegin = max(kbegin, chunk * chunk_keys);
     kend = min(kend, (chunk + 1) * chunk_keys);
-    if (kbegin >= kend) return;   // both blocks of the cluster alike, before any barrier or allocation
+    if (!EXT && kbegin >= kend) return;   // both blocks of the cluster alike, before any barrier or allocation
   }
-  const int kt_all = kbegin / BN, n_all = (kend - 1) / BN - kt_all + 1, n_first = (n_all + 1) / 2;
+  const int kt_all = kbegin / BN;
+  int n_all = (kend - 1) / BN - kt_all + 1;
+  // EXT: n_kept tiles from kept_tile on hold kept keys (below kept_upto) and none of the window; they come first
+  int n_kept = 0, kept_tile = 0, kept_upto = 0;
+  if constexpr (EXT) {
+    kept_upto = kept_end(pos0, window, keep);      // of the tile's first row: no later row keeps fewer
+    if (n_chunks > 1) {
+      kept_tile = chunk * (chunk_keys / BN);
+      kept_upto = min(kept_upto, (chunk + 1) * chunk_keys);
+    }
+    n_kept = max((kept_upto + BN - 1) / BN - kept_tile, 0);
+    if (kbegin < kend) {
+      n_kept = min(n_kept, kt_all - kept_tile);
+    } else {                                        // no key of the window is in this chunk
+      n_all = 0;
+      kend = 0;
+    }
+    n_all += n_kept;
+    if (n_all <= 0) return;                         // both blocks of the cluster alike, before any barrier or allocation
+  }
+  const int n_first = (n_all + 1) / 2;
   // this block's key tiles: the first takes n_first of them, the second the rest (none, if there is only one)
-  const int kt_first = kt_all + (rank ? n_first : 0), n_tiles = rank ? n_all - n_first : n_first;
+  const int first_no = rank ? n_first : 0, n_tiles = rank ? n_all - n_first : n_first;
+  auto tile_at = [&](int j) -> int {                // the key tile that is number j of this block
+    const int no = first_no + j;
+    if constexpr (EXT) return no < n_kept ? kept_tile + no : kt_all + no - n_kept;
+    return kt_all + no;
+  };
   const int* bt = block_table + (size_t)seg * max_blocks;
 
   // keys and values of rows that no copy will fill must be finite: P is zero there, and 0 * NaN is NaN
@@ -281,12 +328,14 @@ paged_prefill_tc5_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
     const int piece = min(ps, BN), pieces_per_tile = BN / piece, piece_shift = 31 - __clz(piece);
     // copies tile j's keys (kv = 0) or values (kv = 1) into their stage; false when the block has given up
     auto load = [&](int j, int kv, int page) -> bool {
-      const int s = kv ? j % STAGES : 0, kt = kt_first + j;   // the keys have one stage
-      // runs of the tile with a key in [kbegin, kend): from the one holding the first such key to the one holding the last
-      const int n_valid = ((min(kend, (kt + 1) * BN) - 1) >> piece_shift) - (max(kbegin, kt * BN) >> piece_shift) + 1;
+      const int s = kv ? j % STAGES : 0, kt = tile_at(j);   // the keys have one stage
       const int p0 = lane * piece, j0 = kt * BN + p0;
       // runs wholly before the window may lie in pages already given back: they are not read
-      const bool mine = lane < pieces_per_tile && j0 < kend && j0 + piece > kbegin;
+      const bool mine = lane < pieces_per_tile && ((j0 < kend && j0 + piece > kbegin) || (EXT && j0 < kept_upto));
+      // runs of the tile with a key in [kbegin, kend): from the one holding the first such key to the one holding the last
+      int n_valid;
+      if constexpr (EXT) n_valid = __popc(__ballot_sync(0xffffffffu, mine));
+      else n_valid = ((min(kend, (kt + 1) * BN) - 1) >> piece_shift) - (max(kbegin, kt * BN) >> piece_shift) + 1;
       unsigned long long* full = kv ? &v_full[s] : &k_full[s];
       int stop = 0;
       if (lane == 0) {
@@ -311,8 +360,9 @@ paged_prefill_tc5_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
     // The page of this lane's run is looked up a tile before it is used: the block table is in global memory, and
     // a lookup inside load() would put its latency between every two tiles.
     auto page_of = [&](int j) -> int {
-      const int j0 = (kt_first + j) * BN + lane * piece;
-      return (j < n_tiles && lane < pieces_per_tile && j0 < kend && j0 + piece > kbegin) ? __ldg(bt + j0 / ps) : 0;
+      const int j0 = tile_at(j) * BN + lane * piece;
+      return (j < n_tiles && lane < pieces_per_tile && ((j0 < kend && j0 + piece > kbegin) || (EXT && j0 < kept_upto)))
+                 ? __ldg(bt + j0 / ps) : 0;
     };
     const int kv = warp == 0 ? 0 : 1;
     int page_now = page_of(0);
@@ -378,7 +428,7 @@ paged_prefill_tc5_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
       rate = rates[h];
     }
     for (int j = 0; j < n_tiles; ++j) {
-      const int j0 = (kt_first + j) * BN;
+      const int j0 = tile_at(j) * BN;
       if constexpr (BIAS) {
         // the four warps meet before the table is overwritten and when it is done; a row that has given up goes on
         // meeting the others
@@ -397,14 +447,45 @@ paged_prefill_tc5_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
 #pragma unroll
         for (int i = 0; i < BN; ++i) v[i] = fmaf(v[i], scale_log2e, -table[r + BN - 1 - i]);
       }
+      if constexpr (EXT) {       // from here on v is in log2 units, capped
+        if (cap > 0.f) {
+          const float to_x = scale_log2e * 0.6931471805599453f / cap, cap2 = cap * 1.4426950408889634f;
+          float big0 = 0.f, big1 = 0.f;
+#pragma unroll
+          for (int i = 0; i < BN; i += 2) {
+            big0 = fmaxf(big0, fabsf(v[i]));
+            big1 = fmaxf(big1, fabsf(v[i + 1]));
+          }
+          // a row's stale columns may hold anything, not-a-numbers too: they only choose the way, and are masked below
+          if (__any_sync(0xffffffffu, !(fmaxf(big0, big1) * to_x <= TANH_POLY_MAX))) {
+#pragma unroll
+            for (int i = 0; i < BN; ++i) v[i] = cap2 * tanh_exp(v[i] * to_x);
+          } else {
+#pragma unroll
+            for (int i = 0; i < BN; ++i) v[i] = cap2 * tanh_poly(v[i] * to_x);
+          }
+        } else {
+#pragma unroll
+          for (int i = 0; i < BN; ++i) v[i] *= scale_log2e;
+        }
+      }
       const bool edge = (j0 + BN - 1 > pos0) || (window != 0 && j0 < first_seen(pos0 + BM - 1, window)) || j0 + BN > kend;
       if (edge) {
         // keys this row may see in this tile: [lo, hi), as columns of the tile
         const int hi = min(min(p + 1, kend) - j0, BN);
         const int lo = max(first_seen(p, window) - j0, 0);
+        if constexpr (EXT) {
+          // a kept tile ends where the row tile's kept keys end; in a tile of the window kept keys may lie before lo
+          const bool kept_only = first_no + j < n_kept;
+          const int kp = (kept_only ? min(keep, kept_upto) : keep) - j0, end = kept_only ? min(kp, BN) : hi;
 #pragma unroll
-        for (int i = 0; i < BN; ++i)
-          if (i < lo || i >= hi) v[i] = -INFINITY;
+          for (int i = 0; i < BN; ++i)
+            if ((i < lo && i >= kp) || i >= end) v[i] = -INFINITY;
+        } else {
+#pragma unroll
+          for (int i = 0; i < BN; ++i)
+            if (i < lo || i >= hi) v[i] = -INFINITY;
+        }
       }
       // four independent chains: a single one would be 64 dependent instructions
       float mx0 = -INFINITY, mx1 = -INFINITY, mx2 = -INFINITY, mx3 = -INFINITY;
@@ -415,7 +496,7 @@ paged_prefill_tc5_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
         mx2 = fmaxf(mx2, v[i + 2]);
         mx3 = fmaxf(mx3, v[i + 3]);
       }
-      const float m_tile = fmaxf(fmaxf(mx0, mx1), fmaxf(mx2, mx3)) * (BIAS ? 1.f : scale_log2e);
+      const float m_tile = fmaxf(fmaxf(mx0, mx1), fmaxf(mx2, mx3)) * (BIAS || EXT ? 1.f : scale_log2e);
       // this tile's buffer of P was read by the products of the tile before the last
       if (j > 1 && !bar_wait(&pv_done[j & 1], ((j - 2) >> 1) & 1)) { atomicExch(error, 16); ok = false; TC5_STOP }
       const bool raise = m_tile > m + RAISE_BY || (m == -INFINITY && m_tile > m);
@@ -445,8 +526,8 @@ paged_prefill_tc5_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
         unsigned pk[4];
 #pragma unroll
         for (int i = 0; i < 4; ++i) {
-          const float e0 = exp2f(BIAS ? v[q8 * 8 + 2 * i] - ref : fmaf(v[q8 * 8 + 2 * i], scale_log2e, -ref)),
-                      e1 = exp2f(BIAS ? v[q8 * 8 + 2 * i + 1] - ref : fmaf(v[q8 * 8 + 2 * i + 1], scale_log2e, -ref));
+          const float e0 = exp2f(BIAS || EXT ? v[q8 * 8 + 2 * i] - ref : fmaf(v[q8 * 8 + 2 * i], scale_log2e, -ref)),
+                      e1 = exp2f(BIAS || EXT ? v[q8 * 8 + 2 * i + 1] - ref : fmaf(v[q8 * 8 + 2 * i + 1], scale_log2e, -ref));
           psum += e0;
           psum1 += e1;
           __nv_bfloat162 b2 = __floats2bfloat162_rn(e0, e1);
@@ -455,7 +536,7 @@ paged_prefill_tc5_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
         *reinterpret_cast<uint4*>(prow + ((q8 ^ (r & 7)) << 4)) = make_uint4(pk[0], pk[1], pk[2], pk[3]);   // swizzled
       }
       l += psum + psum1;
-      if (j0 + BN > kend && r < BN && j0 + r >= kend) {
+      if (j0 + BN > kend && r < BN && j0 + r >= kend && !(EXT && first_no + j < n_kept)) {
         // the last tile: values of keys past the end are whatever the page held; P is zero there, but zero
         // times a NaN left by an earlier owner of the page would still be NaN: this thread clears key row r
         if (!bar_wait(&v_full[j % STAGES], (j / STAGES) & 1)) { atomicExch(error, 13); ok = false; TC5_STOP }   // they have landed
@@ -608,13 +689,13 @@ CBIS_EXPORT int cbis_paged_prefill_tc5(const void* q, int q_ld, int total_rows, 
                                        int max_seg_rows, int n_head, int n_kv_head, int hd, int ps, float scale,
                                        int window, int n_chunks, int chunk_keys, float* partial, const int* positions,
                                        int row0, int n_rows, int* error, void* stream, const float* sinks,
-                                       const float* slopes, const float* rates, int v_heads) {
+                                       const float* slopes, const float* rates, int v_heads, float cap, int keep) {
   if (n_seg <= 0 || max_seg_rows <= 0) return CBIS_OK;
   if (n_chunks < 1 || (n_chunks > 1 && (chunk_keys <= 0 || chunk_keys % tc5::BN || !partial || !positions || n_rows <= 0 ||
                                         ((uintptr_t)partial & 15))))
     return CBIS_ERR_BAD_SIZE;
   if ((hd != 128 && hd != 64) || ps < 8 || ps > 128 || (ps & (ps - 1)) || n_head <= 0 || n_kv_head <= 0 ||
-      (v_heads != 1 && (v_heads != n_kv_head || n_head % v_heads)) || (n_head / v_heads) % n_kv_head || !slopes != !rates)
+      (v_heads != 1 && (v_heads != n_kv_head || n_head % v_heads)) || (n_head / v_heads) % n_kv_head || !slopes != !rates || keep < 0)
     return CBIS_ERR_BAD_SIZE;
   if (q_ld % 8 || out_ld % 8 || ((uintptr_t)q & 15) || ((uintptr_t)kc & 15) || ((uintptr_t)vc & 15) ||
       ((uintptr_t)out & 15) || error == nullptr)
@@ -628,8 +709,12 @@ CBIS_EXPORT int cbis_paged_prefill_tc5(const void* q, int q_ld, int total_rows, 
   st = tc5::make_map(&map_v, vc, cache_rows, hd, hd, ps < tc5::BN ? ps : tc5::BN);
   if (st != CBIS_OK) return st;
   const size_t smem = tc5::smem_bytes(hd) + (rates ? tc5::TABLE * sizeof(float) : 0);
-  auto kern = hd == 128 ? (rates ? tc5::paged_prefill_tc5_kernel<128, true> : tc5::paged_prefill_tc5_kernel<128, false>)
-                        : (rates ? tc5::paged_prefill_tc5_kernel<64, true> : tc5::paged_prefill_tc5_kernel<64, false>);
+  const bool ext = cap > 0.f || (keep > 0 && window != 0);
+  if (ext && rates) return CBIS_ERR_BAD_SIZE;      // the two come in kernels of their own
+  auto kern = hd == 128 ? (rates ? tc5::paged_prefill_tc5_kernel<128, true, false>
+                                 : (ext ? tc5::paged_prefill_tc5_kernel<128, false, true> : tc5::paged_prefill_tc5_kernel<128, false, false>))
+                        : (rates ? tc5::paged_prefill_tc5_kernel<64, true, false>
+                                 : (ext ? tc5::paged_prefill_tc5_kernel<64, false, true> : tc5::paged_prefill_tc5_kernel<64, false, false>));
   cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
   if (e != cudaSuccess) return (int)e;
   e = cudaFuncSetAttribute(kern, cudaFuncAttributePreferredSharedMemoryCarveout, (int)cudaSharedmemCarveoutMaxShared);
@@ -637,11 +722,11 @@ CBIS_EXPORT int cbis_paged_prefill_tc5(const void* q, int q_ld, int total_rows, 
   dim3 grid(2u * (unsigned)((max_seg_rows + tc5::BM - 1) / tc5::BM) * n_head * n_seg * n_chunks);
   e = launch_pdl(kern, grid, dim3(tc5::THREADS), smem, (cudaStream_t)stream, map_q, map_k, map_v, block_table, max_blocks,
                  cu_rows, seg_start, (__nv_bfloat16*)out, out_ld, seg0, n_seg, n_head, n_kv_head, ps,
-                 scale * 1.4426950408889634f, window, n_chunks, chunk_keys, partial, row0, error, sinks, slopes, rates, v_heads);
+                 scale * 1.4426950408889634f, window, n_chunks, chunk_keys, partial, row0, error, sinks, slopes, rates, v_heads, cap, keep);
   if (e == cudaSuccess && n_chunks > 1)
     e = launch_pdl(prefill_merge_kernel<__nv_bfloat16, true>, dim3(n_rows), dim3(128), 0, (cudaStream_t)stream,
                    (const float*)partial, positions, (const int*)nullptr, (__nv_bfloat16*)out, out_ld, row0, n_head, hd, window,
-                   n_chunks, chunk_keys, sinks);
+                   n_chunks, chunk_keys, sinks, keep);
   return (int)e;
 }
 
@@ -650,7 +735,7 @@ CBIS_EXPORT int cbis_paged_prefill_tc5(const void* q, int q_ld, int total_rows, 
 // memory) and what the device's SMs have; negative: a CUDA error.  (The occupancy calls of the runtime answer for
 // whole clusters and count an SM pair once; the profiler's counters show two blocks per SM at work.)
 CBIS_EXPORT int cbis_paged_prefill_tc5_blocks_per_sm() {
-  auto kern = tc5::paged_prefill_tc5_kernel<128, false>;
+  auto kern = tc5::paged_prefill_tc5_kernel<128, false, false>;
   cudaFuncAttributes fa;
   cudaError_t e = cudaFuncGetAttributes(&fa, kern);
   if (e != cudaSuccess) return -(int)e;

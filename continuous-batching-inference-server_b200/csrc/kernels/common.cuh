@@ -23,6 +23,7 @@
 #define CBIS_ACT_SILU 3
 #define CBIS_ACT_SIGMOID 4
 #define CBIS_ACT_RELU2 5      // relu(v)^2
+#define CBIS_ACT_TANH 6
 
 #define CBIS_EXPORT extern "C" __attribute__((visibility("default")))
 
@@ -103,6 +104,15 @@ __device__ __forceinline__ int first_seen(int p, int window) {
   return window > 0 ? max(0, p - window + 1) : (window < 0 ? p - p % (-window) : 0);
 }
 
+// With a window or blocks the first `keep` keys of a sequence may stay visible to every later query: the query at p sees
+// keys [0, kept_end) and [first_seen, p].  The two runs are disjoint; never decreases with p.
+__device__ __forceinline__ int kept_end(int p, int window, int keep) {
+  return window != 0 ? min(keep, first_seen(p, window)) : 0;
+}
+
+// A cap on the scaled scores, cap * tanh(s / cap); cap 0: none.
+__device__ __forceinline__ float capped_score(float s, float cap) { return cap > 0.f ? cap * tanhf(s / cap) : s; }
+
 __device__ __forceinline__ float to_f32(float v) { return v; }
 __device__ __forceinline__ float to_f32(__nv_bfloat16 v) { return __bfloat162float(v); }
 __device__ __forceinline__ void from_f32(float& dst, float v) { dst = v; }
@@ -142,6 +152,7 @@ __device__ __forceinline__ float activate(float v, int act) {
   if (act == CBIS_ACT_SILU) return v * sigmoid_f32(v);
   if (act == CBIS_ACT_SIGMOID) return sigmoid_f32(v);
   if (act == CBIS_ACT_RELU2) return v > 0.f ? v * v : 0.f;
+  if (act == CBIS_ACT_TANH) return tanhf(v);
   if (act == CBIS_ACT_GELU_ERF) return 0.5f * v * (1.0f + erff(v * 0.70710678118654752440f));
   if (act == CBIS_ACT_GELU_TANH) {
     const float c = 0.7978845608028654f;  // sqrt(2/pi)

@@ -14,6 +14,8 @@
 //   per head), then the rotation of every head of q and k, and values blended with another layer's values of the same
 //   token: v <- (1 - lambda) v + lambda v_other.  Each of the three steps is optional.
 //   blend_rows: the last of them alone.
+//   qk_turn_norm: the other order, in place: every head of q and k rotated (pairs i, i + dims / 2, cosine and sine times
+//   `length`), then divided by ITS OWN root mean square and, with weights as wide as one head, multiplied by them.
 #include "common.cuh"
 
 namespace cbis {
@@ -135,6 +137,75 @@ __global__ void qk_prepare_kernel(TT* buf, int ld, int q_off, int q_heads, int k
   }
 }
 
+// A group of L lanes per (row, head); a lane takes up to NU units: a unit is V neighbouring pairs, or V entries of those that
+// pass unrotated.  The head stays in registers between the rotation and its norm and is rounded once.
+template <typename TT, int V>
+struct alignas(sizeof(TT) * V) TurnRun {
+  TT e[V];
+};
+template <typename TT, int V, int NU>
+__global__ void __launch_bounds__(256)
+qk_turn_norm_kernel(TT* buf, int ld, int q_off, int q_heads, int k_off, int k_heads, int width, const float* __restrict__ q_w,
+                    const float* __restrict__ k_w, float eps, const int* positions, const float* __restrict__ freqs, int dims,
+                    float length, int L, int rows) {
+  pdl_trigger();
+  pdl_wait();
+  const int heads = q_heads + k_heads, lane = threadIdx.x & (L - 1);
+  const long long unit = ((long long)blockIdx.x * blockDim.x + threadIdx.x) / L;
+  const bool on = unit < (long long)rows * heads;      // lanes past the end go on with the shuffles
+  const int r = on ? (int)(unit / heads) : 0, h = on ? (int)(unit % heads) : 0;
+  const bool is_q = h < q_heads;
+  TT* b = buf + (size_t)r * ld + (is_q ? q_off + h * width : k_off + (h - q_heads) * width);
+  const float* w = is_q ? q_w : k_w;
+  const float p = (float)positions[r];
+  const int half = dims / 2, n_pairs = half / V, n_units = n_pairs + (width - dims) / V;
+  float x0[NU][V], x1[NU][V], ss = 0.f;
+#pragma unroll
+  for (int i = 0; i < NU; ++i) {
+    const int un = i * L + lane;
+    const bool pair = un < n_pairs, in = on && un < n_units;
+    const int c = pair ? un * V : dims + (un - n_pairs) * V;
+    TurnRun<TT, V> a, d;
+    if (in) a = *reinterpret_cast<const TurnRun<TT, V>*>(b + c);
+    if (in && pair) d = *reinterpret_cast<const TurnRun<TT, V>*>(b + c + half);
+#pragma unroll
+    for (int k = 0; k < V; ++k) {
+      float u = in ? to_f32(a.e[k]) : 0.f, v = 0.f;
+      if (in && pair) {
+        v = to_f32(d.e[k]);
+        float sn, cs;
+        sincosf(p * freqs[c + k], &sn, &cs);
+        cs *= length;
+        sn *= length;
+        const float t = u * cs - v * sn;
+        v = v * cs + u * sn;
+        u = t;
+      }
+      x0[i][k] = u;
+      x1[i][k] = v;
+      ss = fmaf(u, u, fmaf(v, v, ss));
+    }
+  }
+  for (int o = 1; o < L; o <<= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+  const float inv = 1.0f / sqrtf(ss / (float)width + eps);
+#pragma unroll
+  for (int i = 0; i < NU; ++i) {
+    const int un = i * L + lane;
+    const bool pair = un < n_pairs;
+    const int c = pair ? un * V : dims + (un - n_pairs) * V;
+    if (!on || un >= n_units) continue;
+    TurnRun<TT, V> a;
+#pragma unroll
+    for (int k = 0; k < V; ++k) from_f32(a.e[k], x0[i][k] * inv * (w ? w[c + k] : 1.f));
+    *reinterpret_cast<TurnRun<TT, V>*>(b + c) = a;
+    if (pair) {
+#pragma unroll
+      for (int k = 0; k < V; ++k) from_f32(a.e[k], x1[i][k] * inv * (w ? w[c + half + k] : 1.f));
+      *reinterpret_cast<TurnRun<TT, V>*>(b + c + half) = a;
+    }
+  }
+}
+
 // out[r, c] = (1 - lambda) a[r, c] + lambda b[r, c]
 template <typename TT>
 __global__ void blend_rows_kernel(const TT* a, int a_ld, const TT* b, int b_ld, TT* out, int out_ld, float lambda,
@@ -181,6 +252,44 @@ CBIS_EXPORT int cbis_qk_prepare(void* buf, int ld, int q_off, int q_heads, int k
   if (dtype == CBIS_F32) CBIS_QKP(float);
   if (dtype == CBIS_BF16) CBIS_QKP(__nv_bfloat16);
 #undef CBIS_QKP
+  return CBIS_ERR_BAD_DTYPE;
+}
+
+// buf [rows, ld] of the compute type, changed in place: q at columns q_off.. (q_heads x width), k at k_off.. (k_heads x
+// width), heads up to 512 wide; q_w / k_w (may be null): width numbers each; freqs (null with dims 0): dims / 2 numbers.
+CBIS_EXPORT int cbis_qk_turn_norm(void* buf, int ld, int q_off, int q_heads, int k_off, int k_heads, int width,
+                                  const float* q_w, const float* k_w, float eps, const int* positions, const float* freqs,
+                                  int dims, float length, int rows, int dtype, void* stream) {
+  if (rows <= 0 || q_heads + k_heads <= 0) return CBIS_OK;
+  if (q_heads < 0 || k_heads < 0 || width <= 0 || width > 512 || dims < 0 || dims > width || dims % 2 || (dims > 0 && !freqs))
+    return CBIS_ERR_BAD_SIZE;
+  const int esz = dtype == CBIS_F32 ? 4 : 2;
+  const bool by4 = width % 4 == 0 && (dims / 2) % 4 == 0 && ld % 4 == 0 && q_off % 4 == 0 && k_off % 4 == 0 &&
+                   !((uintptr_t)buf & (4 * esz - 1));
+  const int V = by4 ? 4 : 1, units = (dims / 2 + width - dims) / V;
+  int L = 1;
+  while (L < 32 && L < units) L *= 2;
+  const int nu = (units + L - 1) / L;
+  const long long threads = (long long)rows * (q_heads + k_heads) * L;
+  if (threads > (1ll << 38)) return CBIS_ERR_TOO_LARGE;
+  const dim3 grid((unsigned)((threads + 255) / 256));
+  cudaStream_t st = (cudaStream_t)stream;
+#define CBIS_TURN(TT, VV, NU)                                                                                          \
+  return (int)launch_pdl(qk_turn_norm_kernel<TT, VV, NU>, grid, dim3(256), 0, st, (TT*)buf, ld, q_off, q_heads, k_off, \
+                         k_heads, width, q_w, k_w, eps, positions, freqs, dims, length, L, rows)
+#define CBIS_TURN_V(TT)                                                                                                \
+  do {                                                                                                                 \
+    if (V == 4 && nu <= 1) CBIS_TURN(TT, 4, 1);                                                                        \
+    if (V == 4 && nu <= 2) CBIS_TURN(TT, 4, 2);                                                                        \
+    if (V == 4) CBIS_TURN(TT, 4, 4);                                                                                   \
+    if (nu <= 1) CBIS_TURN(TT, 1, 1);                                                                                  \
+    if (nu <= 4) CBIS_TURN(TT, 1, 4);                                                                                  \
+    CBIS_TURN(TT, 1, 16);                                                                                              \
+  } while (0)
+  if (dtype == CBIS_F32) CBIS_TURN_V(float);
+  if (dtype == CBIS_BF16) CBIS_TURN_V(__nv_bfloat16);
+#undef CBIS_TURN_V
+#undef CBIS_TURN
   return CBIS_ERR_BAD_DTYPE;
 }
 

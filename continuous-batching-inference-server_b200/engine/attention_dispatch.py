@@ -18,7 +18,8 @@ positions, counted from position 0: the query sees its own block's keys up to p)
 A mixer may also name (attributes, all optional): ``v_head_dim`` (values of another width than the keys; with one
 cached array for keys and values the values are the first entries of its rows), ``slopes`` (a distance bias per
 head; with ``rates`` it grows with the logarithm of the distance), ``sinks`` (a number per head in the softmax's
-denominator), ``q_temp`` (a query temperature by position) and ``talk`` (the softmax weights are mixed across heads; the
+denominator), ``q_temp`` (a query temperature by position), ``cap`` (a cap on the scaled scores), ``keep_first`` (the first keys
+of a sequence that stay visible behind the window) and ``talk`` (the softmax weights are mixed across heads; the
 mixer may then hand over a gate on the result, element by element).
 ``run_attention`` returns how many columns a head's result takes in ``out``.
 """
@@ -52,8 +53,9 @@ def _general_chunks(ctx, n_head, rows, hd):
 
 
 def _extended(ctx, mixer, qkv, cache, view, out, k_pages, v_pages, k_off, v_off, vd, slopes, sinks, q_temp,
-              rates, v_heads=1, done=0) -> int:
-    """Attention with values of their own width, a distance bias, a sink or a query temperature; with ``v_heads`` =
+              rates, v_heads=1, done=0, cap=0.0, keep=0) -> int:
+    """Attention with values of their own width, a distance bias, a sink, a query temperature, a cap on the scores or kept
+    first keys; with ``v_heads`` =
     n_kv_head every query head over the values of every key/value head (the heads of ``out`` and of the numbers per head
     are then these pairs); rows before ``done`` (0 or the decoding rows) have been taken care of.  bfloat16 with
     widths that are multiples of 8: the decoding rows go to the split-KV decode kernel (up to 256 wide; it stores
@@ -62,7 +64,7 @@ def _extended(ctx, mixer, qkv, cache, view, out, k_pages, v_pages, k_off, v_off,
     a power of two).  32-bit, other sizes: the cache-write
     kernel and the general kernel."""
     T, nd, hd, ps = ctx.n_rows, ctx.n_decode, mixer.head_dim, cache.page_size
-    extra = dict(v_head_dim=vd, slopes=slopes, sinks=sinks, q_temp=q_temp, rates=rates, v_heads=v_heads)
+    extra = dict(v_head_dim=vd, slopes=slopes, sinks=sinks, q_temp=q_temp, rates=rates, v_heads=v_heads, cap=cap, keep=keep)
     n_head = mixer.n_head * v_heads
     o = out[:, :n_head * vd]
     by8 = (qkv.dtype == torch.bfloat16 and hd % 8 == 0 and vd % 8 == 0 and qkv.stride(0) % 8 == 0 and k_off % 8 == 0
@@ -84,12 +86,13 @@ def _extended(ctx, mixer, qkv, cache, view, out, k_pages, v_pages, k_off, v_off,
     if mixer.own_kv:
         ops.kv_write(qkv[r], k_off, v_off, k_pages, v_pages, view.slot_mapping[r], mixer.n_kv_head, hd, ps, v_head_dim=vd)
     tc5 = (tiled and first == nd and hd == vd and hd in (64, 128) and 8 <= ps <= 128 and ops.USE_TCGEN05 and q_temp is None
-           and (slopes is None) == (rates is None) and k_pages is not v_pages and o.data_ptr() % 16 == 0)
+           and (slopes is None) == (rates is None) and not (rates is not None and (cap or keep)) and k_pages is not v_pages and o.data_ptr() % 16 == 0)
     if tc5:          # TMA + tcgen05: takes a sink, a bias that grows with the logarithm of the distance, all value heads
         chunks, partial = _key_chunks(ctx, n_head, nd, T, hd, row_tile=128, blocks_per_tile=2, blocks_per_sm=2, min_chunk=8192)
         ops.paged_prefill_tc5(qkv, k_pages, v_pages, view.block_table, ctx.cu_rows, ctx.seg_start, o, nd, ctx.n_segments - nd,
                               ctx.max_seg_rows, n_head, mixer.n_kv_head, hd, ps, mixer.scale, mixer.window, chunks, partial,
-                              ctx.positions, nd, T - nd, sinks=sinks, slopes=slopes, rates=rates, v_heads=v_heads)
+                              ctx.positions, nd, T - nd, sinks=sinks, slopes=slopes, rates=rates, v_heads=v_heads,
+                              cap=cap, keep=keep)
         return vd
     if tiled:        # q and out keep their full row numbering, the kernel finds its rows through cu_rows
         chunks, partial = _key_chunks(ctx, n_head, first, T, vd)
@@ -147,8 +150,10 @@ def run_attention(ctx, mixer, qkv, cache, view, out, gate=None) -> int:
     v_off = k_off if v_name == k_name else k_off + mixer.d_kv      # one array for both: one column block for both
     vd = int(getattr(mixer, "v_head_dim", 0) or hd)
     slopes, sinks, q_temp, rates = (getattr(mixer, a, None) for a in ("slopes", "sinks", "q_temp", "rates"))
-    if vd != hd or slopes is not None or sinks is not None or q_temp is not None:
-        return _extended(ctx, mixer, qkv, cache, view, out, k_pages, v_pages, k_off, v_off, vd, slopes, sinks, q_temp, rates)
+    cap, keep = float(getattr(mixer, "cap", 0.0)), int(getattr(mixer, "keep_first", 0))
+    if vd != hd or slopes is not None or sinks is not None or q_temp is not None or cap or keep:
+        return _extended(ctx, mixer, qkv, cache, view, out, k_pages, v_pages, k_off, v_off, vd, slopes, sinks, q_temp, rates,
+                         cap=cap, keep=keep)
     _plain(ctx, mixer, qkv, cache, view, out, nd, T, hd, ps, k_pages, v_pages, k_off, v_off)
     return hd
 

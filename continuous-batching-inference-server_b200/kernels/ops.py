@@ -17,7 +17,7 @@ import torch
 from .library import kernels, optional_kernels
 
 F32, BF16 = 0, 1
-ACT = {None: 0, "none": 0, "gelu_erf": 1, "gelu_tanh": 2, "silu": 3, "sigmoid": 4, "relu2": 5}      # relu2: relu(v)^2
+ACT = {None: 0, "none": 0, "gelu_erf": 1, "gelu_tanh": 2, "silu": 3, "sigmoid": 4, "relu2": 5, "tanh": 6}      # relu2: relu(v)^2
 
 _STATUS = {-1: "unsupported dtype", -2: "a size that the kernel does not take",
            -3: "misaligned pointer or stride", -4: "size too large for this kernel"}
@@ -207,20 +207,24 @@ def _next_of(w_nk):
 SMALL_WEIGHT = 1 << 20
 
 
-def gemm_small_m(x, w_nk, bias, act, out, accumulate=False):
+def gemm_small_m(x, w_nk, bias, act, out, accumulate=False, group_n: int = 0, act_from: int = 0):
     """out = act(x @ w_nk^T + bias) for up to 64 rows of bfloat16, 32-bit accumulation (weight streaming).
-    ``accumulate`` (32-bit ``out`` only): the result is added to what ``out`` holds."""
+    ``accumulate`` (32-bit ``out`` only): the result is added to what ``out`` holds.  ``group_n`` > 0 (a multiple of 16):
+    the output's columns come in groups of so many (the last may be narrower), and group i multiplies columns
+    i K .. (i + 1) K - 1 of x, K being the weights' width.  The activation is for columns from ``act_from`` on."""
     _need_cuda(x, w_nk, bias, out)
-    M, K = x.shape
-    N = w_nk.shape[0]
-    assert x.dtype == torch.bfloat16 and w_nk.dtype == torch.bfloat16 and w_nk.is_contiguous() and w_nk.shape[1] == K
+    M = x.shape[0]
+    N, K = w_nk.shape
+    assert x.dtype == torch.bfloat16 and w_nk.dtype == torch.bfloat16 and w_nk.is_contiguous()
+    assert x.shape[1] == (-(-N // group_n) * K if group_n else K)
     assert x.stride(1) == 1 and out.stride(1) == 1 and out.shape == (M, N)
     if accumulate and out.dtype != torch.float32:
         raise KernelError("gemm_small_m: a product is added into a 32-bit matrix only")
     nxt, nbytes = _next_of(w_nk)
     st = kernels().cbis_gemm_small_m_bf16(_ptr(x), c_int(x.stride(0)), _ptr(w_nk), _ptr(bias), _ptr(out),
                                           c_int(out.stride(0)), c_int(M), c_int(N), c_int(K), c_int(ACT[act]),
-                                          c_int(dtype_code(out.dtype)), nxt, nbytes, c_int(1 if accumulate else 0), _stream())
+                                          c_int(dtype_code(out.dtype)), nxt, nbytes, c_int(1 if accumulate else 0), _stream(),
+                                          c_int(group_n), c_int(act_from))
     _check(st, "gemm_small_m", f"M={M} N={N} K={K}")
 
 
@@ -517,7 +521,7 @@ def generic_key_chunks(rows: int, n_head: int, max_context: int, head_dim: int):
 
 def paged_attention_generic(q, k_cache, v_cache, block_table, row_seq, positions, out, n_head, n_kv_head,
                             head_dim, page_size, scale, window=0, chunks=(1, 0), partial=None, v_head_dim=0,
-                            slopes=None, sinks=None, q_temp=None, rates=None, v_heads=1):
+                            slopes=None, sinks=None, q_temp=None, rates=None, v_heads=1, cap: float = 0.0, keep: int = 0):
     """Attention of every row over its request's pages: keys max(0,p-window+1)..p for the query at p.
     ``window`` is one signed number in every attention kernel: 0 every key up to p; w > 0 a sliding window of w keys;
     w < 0 the keys of p's own block of -w positions, p - p mod (-w) .. p, blocks counted from position 0.
@@ -530,7 +534,8 @@ def paged_attention_generic(q, k_cache, v_cache, block_table, row_seq, positions
     1 + coef * ln(floor((p + 1) / every) + 1).  ``rates`` (32-bit, per head, with ``slopes``): the bias is
     slope * ln(1 + rate * (p - j)) instead.  ``v_heads`` = n_kv_head: the launch's head h is query head h / v_heads over
     the values of key/value head h % v_heads (``n_head``, and every array per head, counts these pairs; q holds
-    n_head / v_heads heads)."""
+    n_head / v_heads heads).  ``cap`` > 0: the scaled score s becomes cap * tanh(s / cap) (before a bias).  ``keep`` > 0, with a
+    window or blocks: the first ``keep`` keys of a sequence stay visible to every later query."""
     _need_cuda(q, k_cache, v_cache, block_table, row_seq, positions, out, partial)
     T = q.shape[0]
     if head_dim > ATTENTION_MAX_HEAD_DIM:
@@ -557,7 +562,7 @@ def paged_attention_generic(q, k_cache, v_cache, block_table, row_seq, positions
         _ptr(row_seq), _ptr(positions), _ptr(out), c_int(out.stride(0)), c_int(T), c_int(n_head), c_int(n_kv_head),
         c_int(head_dim), c_int(page_size), c_float(scale), c_int(window), c_int(dtype_code(q.dtype)),
         c_int(n_chunks), c_int(chunk_keys), _ptr(partial), _stream(), c_int(vd), c_int(v_row), _ptr(slopes), _ptr(sinks),
-        c_float(coef), c_int(int(every)), _ptr(rates), c_int(v_heads))
+        c_float(coef), c_int(int(every)), _ptr(rates), c_int(v_heads), c_float(cap), c_int(keep))
     _check(st, "paged_attention_generic", f"T={T} heads={n_head}/{n_kv_head} head_dim={head_dim} page={page_size} "
                                           f"chunks={n_chunks}x{chunk_keys}")
 
@@ -578,12 +583,12 @@ def decode_scratch_floats(rows: int, n_head: int, head_dim: int, nsplit: int) ->
 
 def paged_decode_bf16(qkv, k_off, v_off, k_cache, v_cache, block_table, row_seq, positions, slot_mapping, out,
                       scratch, counters, n_head, n_kv_head, head_dim, page_size, scale, window, nsplit, v_head_dim=0,
-                      slopes=None, sinks=None, q_temp=None, rates=None, v_heads=1):
+                      slopes=None, sinks=None, q_temp=None, rates=None, v_heads=1, cap: float = 0.0, keep: int = 0):
     """Decode attention (one query per row) with the keys split ``nsplit`` ways; with ``k_off >= 0`` the
     current token's key/value are taken from ``qkv`` and stored into the cache by the same kernel.
     ``scratch``: ``decode_scratch_floats`` floats; ``counters``: rows*n_head int32, zero before the
-    first launch (every launch leaves them zero).  ``v_head_dim``, ``slopes``, ``sinks``, ``q_temp``, ``rates``, ``v_heads``: as in
-    ``paged_attention_generic`` (widths multiples of 8 up to 256; the scratch is then sized by the values' width)."""
+    first launch (every launch leaves them zero).  ``v_head_dim``, ``slopes``, ``sinks``, ``q_temp``, ``rates``, ``v_heads``,
+    ``cap``, ``keep``: as in ``paged_attention_generic`` (widths multiples of 8 up to 256; the scratch is then sized by the values' width)."""
     _need_cuda(qkv, k_cache, v_cache, block_table, row_seq, positions, slot_mapping, out, scratch, counters, slopes, sinks)
     rows = qkv.shape[0]
     vd = int(v_head_dim) or head_dim
@@ -603,7 +608,7 @@ def paged_decode_bf16(qkv, k_off, v_off, k_cache, v_cache, block_table, row_seq,
         c_int(out.stride(0)), _ptr(scratch), _ptr(counters), c_int(rows), c_int(n_head), c_int(n_kv_head),
         c_int(head_dim), c_int(page_size), c_float(scale), c_int(window), c_int(nsplit), _stream(),
         c_int(int(v_head_dim)), c_int(v_cache.shape[-1]), _ptr(slopes), _ptr(sinks), c_float(coef), c_int(int(every)),
-        _ptr(rates), c_int(v_heads))
+        _ptr(rates), c_int(v_heads), c_float(cap), c_int(keep))
     _check(st, "paged_decode_bf16", f"rows={rows} heads={n_head}/{n_kv_head} head_dim={head_dim} splits={nsplit}")
 
 
@@ -665,12 +670,12 @@ def decode_mix_bf16(qkv, k_off, v_off, k_cache, v_cache, block_table, row_seq, p
 def paged_prefill_bf16(q, k_cache, v_cache, block_table, cu_rows, seg_start, out, seg0, n_seg, max_seg_rows,
                        n_head, n_kv_head, head_dim, page_size, scale, window=0, chunks=(1, 0), partial=None,
                        positions=None, row0=0, n_rows=0, v_head_dim=0, slopes=None, sinks=None, q_temp=None, rates=None,
-                       v_heads=1):
+                       v_heads=1, cap: float = 0.0, keep: int = 0):
     """Attention of the segments seg0..seg0+n_seg-1 (runs of rows given by ``cu_rows``, first positions
     ``seg_start``) over their pages, on the tensor cores.  Head sizes 16, 32, ... 128, page sizes 2^k.
     With ``v_head_dim`` keys and values may have different widths, multiples of 8 up to 128 (the value pages may be
-    the key pages: a row's first entries are then its values); ``slopes``, ``sinks``, ``q_temp``, ``rates``, ``v_heads``: as
-    in ``paged_attention_generic``.
+    the key pages: a row's first entries are then its values); ``slopes``, ``sinks``, ``q_temp``, ``rates``, ``v_heads``, ``cap``,
+    ``keep``: as in ``paged_attention_generic``.
     ``chunks`` = (n, keys) from ``prefill_key_chunks`` cuts the keys n ways over more blocks (every context of the
     step below n * keys); ``partial`` then holds ``n_rows * n_head * n * (head_dim + 4)`` floats, ``positions`` the
     position of every row, ``row0`` and ``n_rows`` name the rows of these segments."""
@@ -699,7 +704,7 @@ def paged_prefill_bf16(q, k_cache, v_cache, block_table, cu_rows, seg_start, out
         c_int(max_seg_rows), c_int(n_head), c_int(n_kv_head), c_int(head_dim), c_int(page_size), c_float(scale),
         c_int(window), c_int(n_chunks), c_int(chunk_keys), _ptr(partial), _ptr(positions), c_int(row0), c_int(n_rows),
         _stream(), c_int(vd), c_int(v_row), _ptr(slopes), _ptr(sinks), c_float(coef), c_int(int(every)), _ptr(rates),
-        c_int(v_heads))
+        c_int(v_heads), c_float(cap), c_int(keep))
     _check(st, "paged_prefill_bf16", f"segments={n_seg} heads={n_head}/{n_kv_head} head_dim={head_dim} page={page_size} "
                                      f"chunks={n_chunks}x{chunk_keys}")
 
@@ -751,12 +756,13 @@ def paged_prefill_f32(q, k_cache, v_cache, block_table, cu_rows, seg_start, out,
 
 def paged_prefill_tc5(q, k_cache, v_cache, block_table, cu_rows, seg_start, out, seg0, n_seg, max_seg_rows,
                       n_head, n_kv_head, head_dim, page_size, scale, window=0, chunks=(1, 0), partial=None,
-                      positions=None, row0=0, n_rows=0, sinks=None, slopes=None, rates=None, v_heads=1):
+                      positions=None, row0=0, n_rows=0, sinks=None, slopes=None, rates=None, v_heads=1, cap: float = 0.0,
+                      keep: int = 0):
     """The same attention as ``paged_prefill_bf16`` on the tcgen05 tensor cores (TMA operands, S and the output in
     tensor memory).  Head size 64 or 128, page sizes 8..128 (powers of two); ``q`` and ``out`` in full row numbering.
     ``chunks``, ``partial``, ``positions``, ``row0``, ``n_rows`` as for ``paged_prefill_bf16`` (chunks from
     ``prefill_key_chunks`` with two blocks per 128-row tile, two per SM and chunks of at least 8,192 keys);
-    ``sinks``, ``slopes`` with ``rates``, ``v_heads`` as in ``paged_attention_generic``."""
+    ``sinks``, ``slopes`` with ``rates``, ``v_heads``, ``cap`` and ``keep`` (not with ``rates``) as in ``paged_attention_generic``."""
     _need_cuda(q, k_cache, v_cache, block_table, cu_rows, seg_start, out, partial, positions)
     if head_dim not in (64, 128):
         raise KernelError(f"tcgen05 prefill attention: head_dim={head_dim} is neither 64 nor 128")
@@ -777,7 +783,7 @@ def paged_prefill_tc5(q, k_cache, v_cache, block_table, cu_rows, seg_start, out,
         c_int(out.stride(0)), c_int(seg0), c_int(n_seg), c_int(max_seg_rows), c_int(n_head), c_int(n_kv_head),
         c_int(head_dim), c_int(page_size), c_float(scale), c_int(window), c_int(n_chunks), c_int(chunk_keys),
         _ptr(partial), _ptr(positions), c_int(row0), c_int(n_rows), _ptr(tcgen05_error_flag(q.device)), _stream(), _ptr(sinks),
-        _ptr(slopes), _ptr(rates), c_int(v_heads))
+        _ptr(slopes), _ptr(rates), c_int(v_heads), c_float(cap), c_int(keep))
     _check(st, "paged_prefill_tc5", f"segments={n_seg} heads={n_head}/{n_kv_head} page={page_size} chunks={n_chunks}x{chunk_keys}")
 
 
@@ -1115,6 +1121,103 @@ def qk_prepare(buf, q_off, q_heads, k_off, k_heads, width, q_weight, k_weight, e
                                    c_int(v_other.stride(0) if v_other is not None else 0), c_float(blend), c_int(rows),
                                    c_int(dtype_code(buf.dtype)), _stream())
     _check(st, "qk_prepare", f"rows={rows} heads={q_heads}/{k_heads} width={width} rot_dims={rot_dims}")
+
+
+def qk_turn_norm(buf, q_off, q_heads, k_off, k_heads, width, eps, positions, freqs, rot_dims, length: float = 1.0,
+                 q_weight=None, k_weight=None):
+    """Every head of q (``q_heads`` x ``width`` columns of ``buf`` from ``q_off``, in place) and of k: its first ``rot_dims``
+    entries rotated in pairs (entry i with i + rot_dims/2) by position * freqs[i], cosine and sine times ``length``; then
+    the head divided by its own root mean square and, with a weight (``width`` numbers, shared by all heads), multiplied by
+    it.  32-bit arithmetic, one rounding; heads up to 512 wide."""
+    _need_cuda(buf, q_weight, k_weight, positions, freqs)
+    rows = buf.shape[0]
+    assert buf.stride(1) == 1 and positions.dtype == torch.int32 and positions.shape[0] >= rows
+    assert q_off + q_heads * width <= buf.shape[1] and k_off + k_heads * width <= buf.shape[1]
+    for w in (q_weight, k_weight):
+        assert w is None or (w.dtype == torch.float32 and w.numel() == width and w.is_contiguous())
+    assert rot_dims == 0 or (freqs.dtype == torch.float32 and freqs.numel() >= rot_dims // 2 and freqs.is_contiguous())
+    st = kernels().cbis_qk_turn_norm(_ptr(buf), c_int(buf.stride(0)), c_int(q_off), c_int(q_heads), c_int(k_off), c_int(k_heads),
+                                     c_int(width), _ptr(q_weight), _ptr(k_weight), c_float(eps), _ptr(positions), _ptr(freqs),
+                                     c_int(rot_dims), c_float(length), c_int(rows), c_int(dtype_code(buf.dtype)), _stream())
+    _check(st, "qk_turn_norm", f"rows={rows} heads={q_heads}/{k_heads} width={width} rot_dims={rot_dims}")
+
+
+TIME_MIXING_MAX_DIM = 512        # the widest head of the time-mixing kernel (cbis_time_mixing_max_dim())
+TOKEN_SHIFT_MOST = 8             # blends token_shift takes
+
+
+def token_shift(h, state, seg_slot, row_seq, cu_rows, mu, out):
+    """out[:, s * W:(s + 1) * W] = h + (h' - h) * mu[s] with h' the row before each row: the row above it in its segment,
+    or, for a segment's first row, the request's row of ``state`` (32-bit, ``[slots, >= W]``), which then takes the
+    segment's last row.  ``mu`` 32-bit ``[blends, W]``; rows of no segment (``row_seq`` negative) come out as zeros."""
+    _need_cuda(h, state, seg_slot, row_seq, cu_rows, mu, out)
+    rows, W = h.shape
+    n = mu.shape[0]
+    assert h.stride(1) == 1 and out.stride(1) == 1 and out.shape == (rows, n * W) and out.dtype == h.dtype
+    assert mu.dtype == torch.float32 and mu.is_contiguous() and mu.shape[1] == W
+    assert state.dtype == torch.float32 and state.stride(1) == 1 and state.shape[1] >= W
+    assert row_seq.dtype == torch.int32 and row_seq.shape[0] >= rows
+    st = kernels().cbis_token_shift(_ptr(h), c_int(h.stride(0)), _ptr(state), ctypes.c_longlong(state.stride(0)), _ptr(seg_slot),
+                                    _ptr(row_seq), _ptr(cu_rows), _ptr(mu), c_int(n), _ptr(out), c_int(out.stride(0)), c_int(W),
+                                    c_int(rows), c_int(dtype_code(h.dtype)), _stream())
+    _check(st, "token_shift", f"rows={rows} width={W} blends={n}")
+
+
+def linear_blends(x, w_all, n_groups, group_n, tail_act=None):
+    """Products of blends that lie side by side in x (K columns each, K the weights' width): the first ``n_groups`` with
+    ``group_n`` rows of ``w_all`` each, the one after them with the rows left over, through ``tail_act``.  Returns
+    (``[T, n_groups * group_n]``, ``[T, rest]``) of x's type.  A few rows of bfloat16: one weight-streaming product."""
+    _need_cuda(x, w_all)
+    T = x.shape[0]
+    N, K = w_all.shape
+    n_all = n_groups * group_n
+    rest = N - n_all
+    if (x.dtype == torch.bfloat16 and 0 < T <= SMALL_M and group_n % 16 == 0 and 0 < rest <= group_n and K % 8 == 0
+            and x.stride(0) % 8 == 0 and x.data_ptr() % 16 == 0):
+        out = torch.empty((T, N), dtype=x.dtype, device=x.device)
+        gemm_small_m(x, w_all, None, tail_act, out, group_n=group_n, act_from=n_all)
+        return out[:, :n_all], out[:, n_all:]
+    out = torch.empty((T, n_all), dtype=x.dtype, device=x.device)
+    linear_heads(x, w_all[:n_all].view(n_groups, group_n, K), out)
+    return out, linear(x[:, n_groups * K:], w_all[n_all:], None, tail_act)
+
+
+def time_mixing(x, r_off, k_off, v_off, raw, w0, u, state, seg_slot, cu_rows, n_segments, heads, dim, y, max_seg_rows: int = 0,
+                piece_rows=None):
+    """The recurrence o = (S + diag(u) k v^T)^T r, S <- diag(w) S + k v^T, w = exp(-exp(raw + w0)), per head over every
+    segment's rows, from and into the requests' states.  ``x``: the compute type, r, k and v at their column offsets;
+    ``raw``: 32-bit ``[T, heads * dim]``; ``w0``, ``u``: 32-bit, heads * dim numbers; ``y``: 32-bit ``[T, heads * dim]``;
+    ``state``: 32-bit ``[slots, >= heads * dim * dim]``; ``max_seg_rows``: the step's longest segment if known.
+
+    A segment's rows are walked in order.  Where the step's longest segment is long and its blocks are few
+    (``retention_piece_rows``: the same walk, the same policy), segments are cut into pieces that run side by side; against
+    the walk in one piece the results differ by rounding only.  ``piece_rows``: a piece size of one's own (a multiple of
+    16); 0: never cut."""
+    _need_cuda(x, raw, w0, u, state, seg_slot, cu_rows, y)
+    T = x.shape[0]
+    HD = heads * dim
+    assert x.stride(1) == 1 and max(r_off, k_off, v_off) + HD <= x.shape[1]
+    assert raw.dtype == torch.float32 and raw.stride(1) == 1 and raw.shape == (T, HD)
+    assert y.dtype == torch.float32 and y.stride(1) == 1 and y.shape == (T, HD)
+    assert state.dtype == torch.float32 and state.stride(1) == 1 and state.shape[1] >= HD * dim
+    for t in (w0, u):
+        assert t.dtype == torch.float32 and t.numel() == HD and t.is_contiguous()
+    longest = int(max_seg_rows or 0)
+    rows = 0
+    if piece_rows != 0 and longest > 0:
+        rows = int(piece_rows) if piece_rows is not None else retention_piece_rows(longest, n_segments, heads, dim, dim, total_rows=T)
+        assert rows >= 0 and rows % 16 == 0
+    n_pieces, starts, products = 1, None, None
+    if rows and longest > rows:
+        n_pieces = -(-longest // rows)
+        starts = torch.empty((n_segments * n_pieces, HD * dim), dtype=torch.float32, device=x.device)
+        products = torch.empty((n_segments * n_pieces, HD), dtype=torch.float32, device=x.device)
+    st = kernels().cbis_time_mixing(_ptr(x), c_int(x.stride(0)), c_int(r_off), c_int(k_off), c_int(v_off), _ptr(raw),
+                                    c_int(raw.stride(0)), _ptr(w0), _ptr(u), _ptr(state), ctypes.c_longlong(state.stride(0)),
+                                    _ptr(seg_slot), _ptr(cu_rows), _ptr(y), c_int(y.stride(0)), c_int(n_segments), c_int(heads),
+                                    c_int(dim), c_int(dtype_code(x.dtype)), _stream(), c_int(longest), c_int(n_pieces),
+                                    c_int(rows if n_pieces > 1 else 0), _ptr(starts), _ptr(products))
+    _check(st, "time_mixing", f"segments={n_segments} heads={heads} dim={dim} pieces={n_pieces}", launches=3 if n_pieces > 1 else 1)
 
 
 def qk_head_norm(buf, q_off, q_heads, k_off, k_heads, width, q_weight, k_weight, eps):

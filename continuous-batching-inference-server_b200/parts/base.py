@@ -56,10 +56,12 @@ class CacheArray:
 class CacheNeed:
     """What a mixer keeps per token, as a list of named arrays (attention: "k" and "v" of
     ``[n_kv_head, head_dim]``; a mixer with one compressed vector per token: one array of one head).
-    ``window`` 0 keeps every token; w > 0 keeps only what queries at later positions can reach.
+    ``window`` 0 keeps every token; w > 0 keeps only what queries at later positions can reach, and beside it the
+    ``keep_first`` first tokens of a sequence, if the mixer goes on seeing them.
     Layers whose needs are equal share a group: one pool of pages, one block table per request."""
     arrays: Tuple[CacheArray, ...]
     window: int = 0
+    keep_first: int = 0
 
     @staticmethod
     def keys_values(n_kv_head: int, head_dim: int, window: int = 0) -> "CacheNeed":
