@@ -7,6 +7,7 @@ from .figotar import FigotarConfig
 from .vatevik import VatevikConfig
 from .divitar import DivitarConfig
 from .fororax import FororaxConfig
+from .vipovik import VipovikConfig
 
 for _name in ("GPT2LMHeadModel", "TinyGPT", "gpt2"):
     register_architecture(_name, GPT2Config)
@@ -15,6 +16,7 @@ register_architecture("Figotar", FigotarConfig)
 register_architecture("Vatevik", VatevikConfig)
 register_architecture("Divitar", DivitarConfig)
 register_architecture("Fororax", FororaxConfig)
+register_architecture("Vipovik", VipovikConfig)
 
-__all__ = ["ConfigError", "LayerSpec", "ModelSpec", "PartSpec", "GPT2Config", "VekedraConfig", "FigotarConfig", "VatevikConfig", "DivitarConfig", "FororaxConfig", "architecture_name",
+__all__ = ["ConfigError", "LayerSpec", "ModelSpec", "PartSpec", "GPT2Config", "VekedraConfig", "FigotarConfig", "VatevikConfig", "DivitarConfig", "FororaxConfig", "VipovikConfig", "architecture_name",
            "config_from_dict", "known_architectures", "load_config", "register_architecture"]

@@ -50,6 +50,11 @@ class LayerSpec:
     # a constant on the stream before a part's result joins it (1: none), for the arrangements that know it
     stream_scale: float = 1.0
     side: Optional[PartSpec] = None
+    # an earlier layer whose parts (weights) this one runs with, in a block, a cache and a state of its own: the later
+    # passes of layers that run several times.  None: parts of its own
+    weights_from: Optional[int] = None
+    # (index into ModelSpec.pass_inputs, number of the pass) of what stands right ahead of this layer; None: nothing
+    pass_input: Optional[Tuple[int, int]] = None
 
 
 @dataclass(frozen=True)
@@ -70,6 +75,7 @@ class ModelSpec:
     final_norm: PartSpec
     final_norm_prefix: str
     head: Union[None, str, PartSpec]        # the output: logits from the last norm's rows (PartSpec of the head registry)
+    pass_inputs: Tuple[PartSpec, ...] = ()  # what makes a pass's input from the stream (PartSpec of the pass-input registry)
     ignored_tensors: Tuple[str, ...] = ()   # regular expressions of tensors a checkpoint may carry unused
 
     def embedding_spec(self) -> PartSpec:

@@ -55,7 +55,9 @@ __device__ __forceinline__ uint4 ldg_stream(const void* p) {
 // CLUSTER: the kernel is launched in clusters of `ksplit` blocks that share a block's columns and split K.  (A kernel that
 // holds cluster instructions is launched through the cluster scheduler even when it never runs them, which was measured
 // to cost the plain form a third of its speed: the two forms are separate kernels.)
-template <int MT, int NT, int UNROLL, bool LOW8, typename TO, bool CLUSTER = false>
+// GROUP: the output's columns come in groups with columns of A of their own (a form of its own: the parameters would cost the
+// others registers).
+template <int MT, int NT, int UNROLL, bool LOW8, typename TO, bool CLUSTER = false, bool GROUP = false>
 __device__ __forceinline__ void gemm_small_m_body(const __nv_bfloat16* A, int lda, const __nv_bfloat16* __restrict__ W,
                                                   const float* __restrict__ bias, TO* __restrict__ C, int ldc, int M,
                                                   int N, int K, int act, const void* next_w,
@@ -69,7 +71,7 @@ __device__ __forceinline__ void gemm_small_m_body(const __nv_bfloat16* A, int ld
   if constexpr (CLUSTER) rank = (int)cluster_ctarank();
   else ksplit = 1;
   const int n0 = (blockIdx.x / ksplit) * (NT * 8);
-  if (group_n > 0) A += (size_t)(n0 / group_n) * K;      // group_n is a multiple of a block's columns
+  if constexpr (GROUP) A += (size_t)(n0 / group_n) * K;      // group_n is a multiple of a block's columns
   const int nkb_all = (K + 31) / 32;
   const int per_rank = (nkb_all + ksplit - 1) / ksplit;
   const int kb_first = rank * per_rank;
@@ -193,7 +195,7 @@ __device__ __forceinline__ void gemm_small_m_body(const __nv_bfloat16* A, int ld
     if constexpr (CLUSTER)
       for (int r = 1; r < ksplit; ++r) v += others[(size_t)(r - 1) * (MT * 16) * (NT * 8) + idx];
     v += bias0;
-    if (n >= act_from) v = activate(v, act);
+    if (!GROUP || n >= act_from) v = activate(v, act);
     if (accumulate) v += to_f32(C[(size_t)m * ldc + n]);   // C is the residual stream: written by earlier kernels, all behind the wait
     from_f32(C[(size_t)m * ldc + n], v);
   }
@@ -201,12 +203,12 @@ __device__ __forceinline__ void gemm_small_m_body(const __nv_bfloat16* A, int ld
 
 // Two entry points over the same body: the compiler's own register choice for the general form (80 registers,
 // three blocks per SM), and a cap of 64 registers for the M <= 8 form so that four blocks fit.
-template <int MT, int NT, int UNROLL, typename TO>
+template <int MT, int NT, int UNROLL, typename TO, bool GROUP>
 __global__ void __launch_bounds__(SM_WARPS * 32)
 gemm_small_m_kernel(const __nv_bfloat16* A, int lda, const __nv_bfloat16* __restrict__ W,
                     const float* __restrict__ bias, TO* __restrict__ C, int ldc, int M, int N, int K, int act,
                     const void* next_w, unsigned long long next_bytes, int ksplit, int accumulate, int group_n, int act_from) {
-  gemm_small_m_body<MT, NT, UNROLL, false, TO>(A, lda, W, bias, C, ldc, M, N, K, act, next_w, next_bytes, ksplit, accumulate, group_n, act_from);
+  gemm_small_m_body<MT, NT, UNROLL, false, TO, false, GROUP>(A, lda, W, bias, C, ldc, M, N, K, act, next_w, next_bytes, ksplit, accumulate, group_n, act_from);
 }
 template <int MT, int NT, int UNROLL, typename TO>
 __global__ void __launch_bounds__(SM_WARPS * 32, 4)
@@ -231,7 +233,7 @@ static int launch_small_m(const void* A, int lda, const void* W, const float* bi
   void (*kern)(const __nv_bfloat16*, int, const __nv_bfloat16*, const float*, TO*, int, int, int, int, int, const void*,
                unsigned long long, int, int, int, int);
   if constexpr (LOW8) kern = ksplit > 1 ? gemm_small_m_low8_ksplit_kernel<MT, NT, UNROLL, TO> : gemm_small_m_low8_kernel<MT, NT, UNROLL, TO>;
-  else kern = gemm_small_m_kernel<MT, NT, UNROLL, TO>;
+  else kern = group_n > 0 ? gemm_small_m_kernel<MT, NT, UNROLL, TO, true> : gemm_small_m_kernel<MT, NT, UNROLL, TO, false>;
   if (!LOW8 && ksplit > 1) return CBIS_ERR_BAD_SIZE;
   if (smem > 48 * 1024) {
     cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
@@ -277,7 +279,7 @@ static int dispatch_small_m(const void* A, int lda, const void* W, const float* 
   // Few columns and a long K (the feed-forward's second product: 2,048 x 8,192): 8 columns per block would leave
   // each warp 32 K blocks to walk in four dependent rounds.  Then 16 columns per block and K over the 2 or 4 blocks of
   // a cluster, whose sums meet in the first block's shared memory: one round per warp, as many blocks as before.
-  if (M <= 8 && ksplit_enabled() && N < 148 * 2 * 16 && N >= 64) {
+  if (M <= 8 && group_n == 0 && ksplit_enabled() && N < 148 * 2 * 16 && N >= 64) {
     const int tiles16 = (N + 15) / 16, nkb = (K + 31) / 32;
     int ks = 1;
     while (ks < 4 && tiles16 * ks * 2 <= 4 * 148 && nkb >= SM_WARPS * 4 * ks * 2) ks *= 2;
@@ -287,7 +289,7 @@ static int dispatch_small_m(const void* A, int lda, const void* W, const float* 
   // Columns per block: 16 when that still gives the 148 SMs about two blocks each, else 8.
   const bool wide = N >= 148 * 2 * 16;
   // M <= 8 and more 16-column blocks than fit at three per SM (444): the 64-register form runs them in one round
-  if (M <= 8 && wide && (N + 15) / 16 > 3 * 148 && (N + 15) / 16 <= 4 * 148)
+  if (M <= 8 && group_n == 0 && wide && (N + 15) / 16 > 3 * 148 && (N + 15) / 16 <= 4 * 148)
     return launch_small_m<1, 2, 4, true, TO>(A, lda, W, bias, C, ldc, M, N, K, act, next_w, next_bytes, st, accumulate, group_n, act_from);
   if (M <= 16) {
     if (wide) return launch_small_m<1, 2, 4, false, TO>(A, lda, W, bias, C, ldc, M, N, K, act, next_w, next_bytes, st, accumulate, group_n, act_from);

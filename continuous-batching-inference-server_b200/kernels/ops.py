@@ -211,7 +211,7 @@ def gemm_small_m(x, w_nk, bias, act, out, accumulate=False, group_n: int = 0, ac
     """out = act(x @ w_nk^T + bias) for up to 64 rows of bfloat16, 32-bit accumulation (weight streaming).
     ``accumulate`` (32-bit ``out`` only): the result is added to what ``out`` holds.  ``group_n`` > 0 (a multiple of 16):
     the output's columns come in groups of so many (the last may be narrower), and group i multiplies columns
-    i K .. (i + 1) K - 1 of x, K being the weights' width.  The activation is for columns from ``act_from`` on."""
+    i K .. (i + 1) K - 1 of x, K being the weights' width.  With groups the activation is for columns from ``act_from`` on."""
     _need_cuda(x, w_nk, bias, out)
     M = x.shape[0]
     N, K = w_nk.shape

@@ -14,7 +14,8 @@ import torch
 
 from ..config import ModelSpec, load_config
 from ..kernels import ops
-from ..parts import (make_block, make_embedding, make_feed_forward, make_head, make_mixer, make_norm, make_position)
+from ..parts import (make_block, make_embedding, make_feed_forward, make_head, make_mixer, make_norm, make_pass_input,
+                     make_position)
 from ..weights import TensorDecl, check_tensors, read_model_tensors
 
 _DTYPES = {"bfloat16": torch.bfloat16, "bf16": torch.bfloat16, "float32": torch.float32, "fp32": torch.float32,
@@ -30,8 +31,15 @@ def resolve_dtype(dtype) -> torch.dtype:
 class Layer:
     """A block with its parts and the tensor-name prefix of its weights."""
 
-    def __init__(self, spec, index: int):
-        self.spec, self.index = spec, index
+    def __init__(self, spec, index: int, shared: Optional["Layer"] = None):
+        """``shared``: the layer whose parts this one runs with (``LayerSpec.weights_from``)."""
+        self.spec, self.index, self.shares = spec, index, shared is not None
+        if shared is not None:
+            for name in ("mixer", "feed_forward", "norm_mixer", "norm_feed_forward", "post_norm_mixer",
+                         "post_norm_feed_forward", "side"):
+                setattr(self, name, getattr(shared, name))
+            self._make_block(spec)
+            return
         extra = {"own_kv": False} if spec.cache_source is not None and spec.mixer.kind == "attention" else {}
         self.mixer = make_mixer(spec.mixer, **extra)
         self.feed_forward = make_feed_forward(spec.feed_forward)
@@ -41,6 +49,9 @@ class Layer:
         self.post_norm_feed_forward = (make_norm(spec.post_norm_feed_forward)
                                        if spec.post_norm_feed_forward is not None else None)
         self.side = make_feed_forward(spec.side) if spec.side is not None else None
+        self._make_block(spec)
+
+    def _make_block(self, spec):
         extra = {}
         if spec.residual_scale != 1.0 or self.side is not None:
             extra = {"residual_scale": spec.residual_scale, "side": self.side}
@@ -52,6 +63,8 @@ class Layer:
         self.post_norm_names = tuple(spec.post_norm_prefixes)
 
     def parts(self):
+        if self.shares:         # they are listed, loaded and counted with the layer they belong to
+            return []
         p = self.spec.prefix
         out = [(p, self.mixer), (p, self.feed_forward), (p + self.norm_names[0], self.norm_mixer),
                (p + self.norm_names[1], self.norm_feed_forward)]
@@ -72,7 +85,16 @@ class Model:
         self.spec = spec
         self.embedding = make_embedding(spec.embedding_spec())
         self.position = make_position(spec.position)
-        self.layers: List[Layer] = [Layer(ls, i) for i, ls in enumerate(spec.layers)]
+        self.layers: List[Layer] = []
+        for i, ls in enumerate(spec.layers):
+            src = ls.weights_from
+            if src is not None and not (0 <= src < i and not self.layers[src].shares):
+                raise ValueError(f"layer {i} runs with the weights of layer {src}, which is no earlier layer with weights of its own")
+            self.layers.append(Layer(ls, i, None if src is None else self.layers[src]))
+        self.pass_inputs = [make_pass_input(p) for p in spec.pass_inputs]
+        for ls in spec.layers:
+            if ls.pass_input is not None and not 0 <= ls.pass_input[0] < len(self.pass_inputs):
+                raise ValueError(f"layer {ls.prefix!r} names pass input {ls.pass_input[0]}, which does not exist")
         for i in spec.schedule:
             if not 0 <= i < len(self.layers):
                 raise ValueError(f"schedule names layer {i}; the model has {len(self.layers)} layers")
@@ -95,7 +117,7 @@ class Model:
 
     def all_parts(self):
         """(tensor-name prefix, part) of every part of the model, in loading order."""
-        out = [("", self.embedding), ("", self.position)]
+        out = [("", self.embedding), ("", self.position)] + [("", p) for p in self.pass_inputs]
         for layer in self.layers:
             out += layer.parts()
         return out + [(self.spec.final_norm_prefix, self.final_norm), ("", self.head_part)]
@@ -125,6 +147,8 @@ class Model:
         order = []
         for li in self.spec.schedule:
             layer = self.layers[li]
+            if layer.spec.pass_input is not None:
+                order += self.pass_inputs[layer.spec.pass_input[0]].streamed_weights()
             order += layer.mixer.streamed_weights() + layer.feed_forward.streamed_weights()
             if layer.side is not None:
                 order += layer.side.streamed_weights()
@@ -142,7 +166,7 @@ class Model:
         for _, part in self.all_parts():
             if part is self.embedding or part is self.position:
                 continue
-            for v in vars(part).values():
+            for v in (part.step_weights() if hasattr(part, "step_weights") else vars(part).values()):
                 add(v)
         return total
 
@@ -151,11 +175,16 @@ class Model:
         """Logits (float32 ``[R, vocab]``) at ``ctx.logit_rows`` for the rows of this step."""
         ctx.shared = {}      # what layers hand to later layers within one step
         x = self.embedding.forward(ctx, self.position)
+        for p in self.pass_inputs:
+            p.begin(ctx, x)
         pending = None
         sched = self.spec.schedule
         i = 0
         while i < len(sched):
             li = sched[i]
+            ahead = self.layers[li].spec.pass_input
+            if ahead is not None:
+                x, pending = self.pass_inputs[ahead[0]].forward(ctx, x, pending, ahead[1])
             block, cache, state = self.layers[li].block, ctx.layer_cache(li), ctx.layer_state(li)
             key = block.run_key(ctx, cache, state)
             if key is None:
@@ -168,7 +197,7 @@ class Model:
             while j < len(sched):
                 nxt = self.layers[sched[j]].block
                 c2, s2 = ctx.layer_cache(sched[j]), ctx.layer_state(sched[j])
-                if type(nxt) is not type(block) or nxt.run_key(ctx, c2, s2) != key:
+                if self.layers[sched[j]].spec.pass_input is not None or type(nxt) is not type(block) or nxt.run_key(ctx, c2, s2) != key:
                     break
                 run.append((nxt, c2, s2))
                 j += 1
@@ -184,7 +213,10 @@ def declared_tensors(spec: ModelSpec) -> List[TensorDecl]:
 def load_model(folder: str, dtype="bfloat16", device="cuda") -> Model:
     """Model of ``folder`` (config.json chooses the architecture; model.safetensors by tensor name)."""
     config = load_config(folder)
+    tensors = read_model_tensors(folder)
+    if hasattr(config, "with_shapes"):      # a format may leave a size to a tensor's shape
+        config = config.with_shapes({name: tuple(t.shape) for name, t in tensors.items()})
     model = Model(config.model_spec())
     model.config = config
-    model.load(read_model_tensors(folder), dtype, device, where=f"{folder}/model.safetensors")
+    model.load(tensors, dtype, device, where=f"{folder}/model.safetensors")
     return model

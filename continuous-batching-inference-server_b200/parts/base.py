@@ -5,7 +5,7 @@ declares the tensors it needs under a name prefix, takes them at load time, and 
 run by a block with a ``StepContext``.  No part knows which model or which layer it
 is in.  New kinds are added with ``register_mixer`` / ``register_feed_forward`` /
 ``register_norm`` / ``register_position`` / ``register_block`` / ``register_embedding`` /
-``register_head``; a configuration then names them in its ``ModelSpec``.  A part refuses sizes
+``register_head`` / ``register_pass_input``; a configuration then names them in its ``ModelSpec``.  A part refuses sizes
 that no kernel takes in its constructor, so a model that cannot run fails when it is built.
 
 Values that flow between parts:
@@ -145,6 +145,19 @@ class Mixer(Part):
         (the 32-bit rows, set while a block runs its parts), which a part is free to ignore."""
         raise NotImplementedError
 
+    # Optional: a mixer whose last step is one plain product, ``w_out`` ``[width, heads_width]``, may offer the rows that go
+    # into it, for a part that runs the last steps of several mixers as one product (``SideBySide``).  A mixer with
+    # ``scales_heads`` multiplies its rows by a constant at no cost (``scale_heads``, before it runs).
+    heads_width = 0
+    scales_heads = False
+
+    def scale_heads(self, factor: float) -> None:
+        raise NotImplementedError
+
+    def forward_heads(self, ctx, h: torch.Tensor, cache, state: Optional[torch.Tensor], out: torch.Tensor) -> None:
+        """Writes the rows ``[T, heads_width]`` (compute dtype, maybe a view of wider rows) into ``out``."""
+        raise NotImplementedError
+
     # Optional: a mixer may take the residual stream itself, normalise it inside its first kernel and add its result
     # into it.  A block asks ``fuses_norm`` every step and calls ``forward_residual`` only after a yes.
     def fuses_norm(self, ctx, norm: "Norm") -> bool:
@@ -221,6 +234,19 @@ class Embedding(Part):
     table: Optional[torch.Tensor] = None
 
     def forward(self, ctx, position: PositionEncoding) -> torch.Tensor:
+        raise NotImplementedError
+
+
+class PassInput(Part):
+    """What stands ahead of every pass of layers that run several times: makes the stream the pass begins with from the
+    stream as it is and from the embedding's output."""
+
+    def begin(self, ctx, x: torch.Tensor) -> None:
+        """Called once a step with the embedding's output, before any layer changes it."""
+
+    def forward(self, ctx, x: torch.Tensor, pending: Optional[Delta], number: int) -> Tuple[torch.Tensor, Optional[Delta]]:
+        """The stream (32-bit rows) of pass ``number`` and what is still to be added to it; ``pending``: what the layer
+        before left to be added to x."""
         raise NotImplementedError
 
 
@@ -314,6 +340,7 @@ _POSITIONS: Dict[str, Callable[..., PositionEncoding]] = {}
 _BLOCKS: Dict[str, Callable[..., Block]] = {}
 _EMBEDDINGS: Dict[str, Callable[..., Embedding]] = {}
 _HEADS: Dict[str, Callable[..., Head]] = {}
+_PASS_INPUTS: Dict[str, Callable[..., PassInput]] = {}
 
 
 def register_mixer(kind: str, factory) -> None:
@@ -344,6 +371,10 @@ def register_head(kind: str, factory) -> None:
     _HEADS[kind] = factory
 
 
+def register_pass_input(kind: str, factory) -> None:
+    _PASS_INPUTS[kind] = factory
+
+
 def _make(table, what, spec, **extra):
     if spec.kind not in table:
         raise KeyError(f"unknown {what} kind {spec.kind!r}; known: {sorted(table)}")
@@ -368,6 +399,10 @@ def make_position(spec) -> PositionEncoding:
 
 def make_embedding(spec) -> Embedding:
     return _make(_EMBEDDINGS, "embedding", spec)
+
+
+def make_pass_input(spec) -> PassInput:
+    return _make(_PASS_INPUTS, "pass input", spec)
 
 
 def make_head(spec) -> Head:

@@ -7,7 +7,7 @@ import torch
 from ..kernels import ops
 from ..weights.loader import TensorDecl
 from .base import CacheArray, CacheNeed, Delta, Mixer, register_mixer
-from .rotation import rotary_frequencies
+from .rotation import blended_frequencies, rotary_frequencies
 
 
 class RotaryAttention(Mixer):
@@ -34,6 +34,13 @@ class RotaryAttention(Mixer):
     * ``block`` > 0: the query at position p sees only the keys of its own block of ``block`` positions, those from
       p - p mod block on, blocks counted from position 0 of the sequence however a prompt was cut (instead of a
       sliding ``window``; the kernels take both in one signed number, ``mask``).
+    * ``rot_blend`` = (factor, original, fast, slow): the slow pairs are slowed down and cosines and sines lengthened
+      (``parts.rotation.blended_frequencies``).
+    * ``turned_norm``: every head of q and of k is divided by its own root mean square (``eps``, no weight) AFTER its
+      rotation; keys are cached so.
+    * ``cap`` > 0: the score becomes cap * tanh(score / cap).
+    * ``keep_first`` > 0, with a window: the first ``keep_first`` keys of a sequence stay visible behind it, at their true
+      positions; the cache keeps their pages.
     * ``head_gate``: head h's output is multiplied by sigmoid of one number per token and head, a projection of the
       mixer's input (``<gate>``, no bias).
 
@@ -45,7 +52,8 @@ class RotaryAttention(Mixer):
                  window: int = 0, qk_norm: bool = False, eps: float = 1e-5, rot_base: float = 10000.0, rot_dims: int = 0,
                  rot_stretch=None, unit_sink: bool = False, value_blend: str = None,
                  names=("mix.q", "mix.k", "mix.v", "mix.o", "mix.vmix", "mix.g"), bias: bool = False,
-                 values_from_keys: bool = False, rot_divide: float = 1.0, block: int = 0, head_gate: bool = False):
+                 values_from_keys: bool = False, rot_divide: float = 1.0, block: int = 0, head_gate: bool = False,
+                 rot_blend=None, turned_norm: bool = False, cap: float = 0.0, keep_first: int = 0):
         if n_head % n_kv_head:
             raise ValueError(f"n_head={n_head} is not a multiple of n_kv_head={n_kv_head}")
         for what, v in (("head_dim", head_dim), ("v_head_dim", v_head_dim)):
@@ -72,8 +80,19 @@ class RotaryAttention(Mixer):
         if self.rot_dims % 2 or not 0 <= self.rot_dims <= self.head_dim:
             raise ValueError(f"rot_dims={self.rot_dims} must be even and at most head_dim={self.head_dim}")
         self.rot_stretch = None if rot_stretch is None else tuple(float(v) for v in rot_stretch)
+        self.rot_blend = None if rot_blend is None else tuple(float(v) for v in rot_blend)
+        if self.rot_blend is not None and (self.rot_stretch is not None or self.rot_divide != 1.0):
+            raise ValueError("rot_blend goes with neither rot_stretch nor rot_divide")
+        self.rot_length = 1.0
+        self.turned_norm, self.cap, self.keep_first = bool(turned_norm), float(cap), int(keep_first)
+        if (self.turned_norm or self.rot_blend is not None) and (self.qk_norm or self.values_from_keys or value_blend == "blend"):
+            raise ValueError("turned_norm and rot_blend go with neither a norm over the projections, nor values taken from the "
+                             "keys, nor blended values")
+        if self.cap < 0 or self.keep_first < 0 or (self.keep_first and not self.window):
+            raise ValueError(f"cap={cap} and keep_first={keep_first} must not be negative, and keep_first needs a window")
         self.unit_sink, self.value_blend = bool(unit_sink), value_blend
         self.d_q, self.d_kv, self.d_v = self.n_head * self.head_dim, self.n_kv_head * self.head_dim, self.n_kv_head * self.v_head_dim
+        self.heads_width = self.n_head * self.v_head_dim
         # wider rows than the kernel that prepares q and k in one pass holds: the same in kernels of their own
         self.one_pass = self.d_q + self.d_kv <= ops.QK_PREPARE_MAX_WIDTH
         defaults = ("mix.q", "mix.k", "mix.v", "mix.o", "mix.vmix", "mix.g")
@@ -84,7 +103,7 @@ class RotaryAttention(Mixer):
     def cache_need(self):
         # behind a sliding window pages go back; blocks keep theirs (0: nothing is given back)
         return CacheNeed((CacheArray("k", self.n_kv_head, self.head_dim), CacheArray("v", self.n_kv_head, self.v_head_dim)),
-                         max(self.window, 0))
+                         max(self.window, 0), self.keep_first if self.window > 0 else 0)
 
     def _inputs(self):
         """(tensor name, rows, has a bias) of the matrices that form the one input product, in its column order."""
@@ -124,7 +143,11 @@ class RotaryAttention(Mixer):
             self.q_norm_w, self.k_norm_w = self._vector(tensors[n[0] + ".norm"], device), self._vector(tensors[n[1] + ".norm"], device)
         if self.value_blend == "blend":
             self.blend = float(tensors[n[4]].to(torch.float32).reshape(()).item())      # a constant of the model
-        self.freqs = rotary_frequencies(self.rot_base, self.rot_dims, self.rot_stretch, self.rot_divide).to(device)
+        if self.rot_blend is not None:
+            table, self.rot_length = blended_frequencies(self.rot_base, self.rot_dims, *self.rot_blend)
+        else:
+            table = rotary_frequencies(self.rot_base, self.rot_dims, self.rot_stretch, self.rot_divide)
+        self.freqs = table.to(device)
         if self.unit_sink:      # a sink of score 0: exp(0) joins the denominator
             self.sinks = torch.zeros(self.n_head, dtype=torch.float32, device=device)
 
@@ -132,13 +155,20 @@ class RotaryAttention(Mixer):
         return [self.w_in, self.w_out]
 
     def forward(self, ctx, h, cache, state):
+        out = torch.empty((h.shape[0], self.heads_width), dtype=h.dtype, device=h.device)
+        self.forward_heads(ctx, h, cache, state, out)
+        if ops.linear_residual(out, self.w_out, ctx.residual):
+            return None
+        return Delta(ops.linear(out, self.w_out, None, None, out_dtype=torch.float32))
+
+    def forward_heads(self, ctx, h, cache, state, out):
         if cache is None:
             raise RuntimeError("attention needs a cache")
         T = h.shape[0]
         k0, v0 = self.d_q, self.d_q + self.d_kv
         proj = ops.linear(h, self.w_in, self.b_in)
         if self.values_from_keys:
-            return self._finish(ctx, h, cache, self._keys_as_values(ctx, proj), proj)
+            return self._finish(ctx, cache, self._keys_as_values(ctx, proj), proj, out)
         other = None
         if self.value_blend == "source":
             ctx.shared["value_blend_source"] = proj[:, v0:v0 + self.d_v]       # stays as projected: this layer blends nothing
@@ -147,7 +177,10 @@ class RotaryAttention(Mixer):
             if other is None or other.shape != (T, self.d_v):
                 raise RuntimeError("a layer that blends its values needs an earlier layer of the step that left values "
                                    f"of the same shape [{T}, {self.d_v}]")
-        if ops.USE_QK_PREPARE and self.one_pass:
+        if self.turned_norm:
+            ops.qk_turn_norm(proj, 0, self.n_head, k0, self.n_kv_head, self.head_dim, self.eps, ctx.positions, self.freqs,
+                             self.rot_dims, self.rot_length)
+        elif self.rot_length == 1.0 and ops.USE_QK_PREPARE and self.one_pass:
             if self.qk_norm or self.rot_dims or other is not None:
                 ops.qk_prepare(proj, 0, self.n_head, k0, self.n_kv_head, self.head_dim, self.q_norm_w, self.k_norm_w,
                                self.eps, ctx.positions, self.freqs, self.rot_dims, v0, self.d_v, other, self.blend)
@@ -158,12 +191,12 @@ class RotaryAttention(Mixer):
                 ops.rms_norm(k, self.k_norm_w, self.eps, k)
             if self.rot_dims:
                 ops.rope_rows(proj, 0, self.head_dim, proj, 0, self.head_dim, ctx.positions, self.n_head, self.head_dim,
-                              self.rot_dims, self.freqs)
+                              self.rot_dims, self.freqs, length=self.rot_length)
                 ops.rope_rows(proj, k0, self.head_dim, proj, k0, self.head_dim, ctx.positions, self.n_kv_head,
-                              self.head_dim, self.rot_dims, self.freqs)
+                              self.head_dim, self.rot_dims, self.freqs, length=self.rot_length)
             if other is not None:
                 ops.blend_rows(v, other, self.blend, v)
-        return self._finish(ctx, h, cache, proj, proj)
+        self._finish(ctx, cache, proj, proj, out)
 
     def _keys_as_values(self, ctx, proj):
         """q | k | v for the attention kernels from the product's q | k: q and k rotated, and the keys as they were
@@ -174,16 +207,11 @@ class RotaryAttention(Mixer):
                       keep_col0=self.d_q + self.d_kv, keep_head0=self.n_head)
         return qkv
 
-    def _finish(self, ctx, h, cache, qkv, proj):
-        T = h.shape[0]
-        out = torch.empty((T, self.n_head * self.v_head_dim), dtype=h.dtype, device=h.device)
+    def _finish(self, ctx, cache, qkv, proj, out):
         ctx.attention(self, qkv, cache, ctx.groups[cache.group], out)     # stores k and v, then attends
         if self.head_gate:
             g0 = proj.shape[1] - self.n_head
             ops.head_gate_mul(out, proj[:, g0:g0 + self.n_head], self.n_head, out)
-        if ops.linear_residual(out, self.w_out, ctx.residual):
-            return None
-        return Delta(ops.linear(out, self.w_out, None, None, out_dtype=torch.float32))
 
 
 register_mixer("rotary_attention", RotaryAttention)
