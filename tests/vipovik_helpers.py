@@ -115,17 +115,22 @@ def make_weights(cfgd, seed, std=0.25, tweak=None):
         if t.dim() == 2 and name != "embed" and not name.endswith((".u", "loop.step")):
             t.mul_((W / t.shape[1]) ** 0.5)         # keep activations of order one
         if name == "loop.in":
-            t.mul_(0.5)
+            t.mul_(0.3)
         if name == "embed":
             t.mul_(3.0)
         if ".mu." in name:
-            t.mul_(1.5).add_(0.5)                   # blends of every kind, beyond both ends too
+            t.add_(0.5)                             # blends of every kind, beyond both ends too
         if name.endswith(".w0"):
             t.mul_(5.0).sub_(2.0)                   # decays from a few tokens to hundreds
-        if name.endswith(".u"):
-            t.mul_(4.0)
         if name.endswith(".router"):
             t.mul_(3.0)                             # scores apart from one another: few close calls
+    for name in [n for n in tensors if n.endswith("right.u")]:
+        # keys that resemble the receptances, positive bonuses: a head's result is divided by its own size, and one that
+        # happens to be near zero (at the first token: r . (u k) near zero) would turn with rounding
+        stem = name[:-1]
+        tensors[name].mul_(3.0).abs_().add_(0.3)
+        tensors[stem + "k"] = 0.85 * tensors[stem + "r"] + 0.5 * tensors[stem + "k"]
+        tensors[stem + "mu.k"] = tensors[stem + "mu.r"] + 0.3 * (tensors[stem + "mu.k"] - tensors[stem + "mu.r"])
     if tweak is not None:
         tweak(tensors)
     return {k: v.to(torch.bfloat16).float() for k, v in tensors.items()}
