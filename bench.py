@@ -116,7 +116,7 @@ def main() -> int:
     ap.add_argument("--warmup", type=int, default=16)
     ap.add_argument("--impl", default="b200", choices=["b200", "reference"])
     ap.add_argument("--config", default="1.3b", choices=["1.3b", "6.7b", "xl", "batching", "vekedra", "figotar", "vatevik", "divitar",
-                                                         "fororax"],
+                                                         "fororax", "vipovik"],
                     help="1.3b: the default measurement; 6.7b: batch-64 decode at context 2,048; "
                          "xl: 64 mixed requests through the scheduler (prompts 32-768, 256 outputs each); "
                          "batching: the reference's own workload at the reference's own sizes (both --impl arms); "
@@ -125,7 +125,8 @@ def main() -> int:
                          "figotar: the same for the Figotar design, beside Vekedra and the GPT-2 style model; "
                          "vatevik: the same for the Vatevik design, beside Figotar and the GPT-2 style model; "
                          "divitar: the same for the Divitar design, beside Figotar, Vekedra and the GPT-2 style model; "
-                         "fororax: the same for the Fororax design, beside Divitar, Vatevik and the GPT-2 style model")
+                         "fororax: the same for the Fororax design, beside Divitar, Vatevik and the GPT-2 style model; "
+                         "vipovik: the same for the Vipovik design, beside Vatevik, Fororax and the GPT-2 style model")
     ap.add_argument("--batch", type=int, default=None)
     ap.add_argument("--prompt-len", type=int, default=None)
     ap.add_argument("--layers", type=int, default=None, help="run fewer layers than the configuration has")
@@ -168,6 +169,8 @@ def main() -> int:
         return divitar_workload(args, cb, torch)
     if args.config == "fororax":
         return fororax_workload(args, cb, torch)
+    if args.config == "vipovik":
+        return vipovik_workload(args, cb, torch)
     if args.config == "6.7b":
         args.skip_points = True
         args.batch = args.batch or 64
@@ -1111,6 +1114,203 @@ def fororax_kernels(torch, ops, pk):
     timed(decode(mixing=True), nbytes, "attention_decode_8_mixed_heads")
     timed(decode(v_heads=nkv, sinks=every), nbytes, "attention_decode_8_mixed_heads_every_head_over_every_value_head")
     timed(decode(sinks=sinks), nbytes, "closest_model_attention_decode_8_sink")
+    return out
+
+
+def vipovik_sizes(width, layers):
+    """A Vipovik configuration whose layer runs have the sizes a model of this width would have: attention (grouped
+    key/value heads, slowed rotation, a cap, a window that keeps the first 16 tokens) beside time mixing with heads of 64, dense
+    and routed feed-forwards in turn; two of the layers run twice, so ``layers`` runs are ``layers`` - 2 layers' weights."""
+    big = width >= 2048
+    hd = 128 if big else 64
+    heads = width // hd
+    mixer = {"left": {"dim": hd, "heads": heads, "kv_heads": max(1, heads // 4), "vdim": hd, "scale": hd ** -0.5, "softcap": 50.0,
+                      "mask": {"size": 1024 if big else 512, "keep_first": 16},
+                      "rot": {"base": 500000.0, "dims": hd, "scaling": {"factor": 8.0, "original": 4096, "fast": 32.0, "slow": 1.0}}},
+             "right": {"dim": 64, "heads": width // 64, "decay_rank": 64}, "left_scale": 0.9, "right_scale": 0.7}
+    dense = {"kind": "dense", "ff": 4 * width}
+    moe = {"kind": "moe", "expert": {"ff": 11 * width // 16, "limit": 7.0}, "router": {"experts": 16 if big else 8, "top": 2}}
+    out = [{"type": "parallel", "mixer": mixer, "mlp": dict(dense if i % 2 == 0 else moe)} for i in range(layers - 2)]
+    return {"architecture": "Vipovik", "embedding": {"scale": 8.0}, "layers": out, "loop": {"start": 2, "stop": 4, "times": 2},
+            "norm": {"eps": 1e-6}, "vocab": 32000, "width": width}
+
+
+def vipovik_workload(args, cb, torch) -> int:
+    """Prefill (one 2,048-token prompt in one step) and decode (batch 8 from context 1,024, the captured step with
+    argmax on the device) of the Vipovik design at two layer sizes, each beside Vatevik (the closest model in its mixers: a
+    matrix recurrence walked row by row, attention with rotated keys; one of the two a layer where Vipovik has both), Fororax
+    (the closest in its routed experts) and the GPT-2 style model of equal width and number of layer runs; then the design's
+    own kernels alone, at the larger size, beside the like kernels of those models."""
+    from cbis_b200.kernels import ops
+    pk = peaks()
+    P, T, B = 2048, 2048, args.batch or 8
+    steps, warm = min(args.steps, 128), max(3, min(args.warmup, 8))
+    layers = max(6, args.layers or 8)
+    gen = torch.Generator().manual_seed(0)
+    sampler = ClockSampler()
+    sampler.start()
+    sizes = {}
+    for width in (1024, 2048):
+        gpt = dict(architectures=["GPT2LMHeadModel"], model_type="gpt2", n_layer=layers, n_embd=width, n_head=16,
+                   n_inner=4 * width, vocab_size=32000, n_positions=P, activation_function="gelu",
+                   layer_norm_epsilon=1e-5, tie_word_embeddings=False)
+        sizes[f"width_{width}"] = {name: measure_model(args, cb, torch, pk, cfgd, 32000, B, P, T, steps, warm, gen)
+                                   for name, cfgd in (("vipovik", vipovik_sizes(width, layers)),
+                                                      ("vatevik", vatevik_sizes(width, layers)),
+                                                      ("fororax", fororax_sizes(width, layers, P)), ("gpt2_style", gpt))}
+    clocks = sampler.stop()
+    line = {"metric": f"Vipovik prefill and decode tokens/s beside Vatevik, Fororax and the GPT-2 style model of equal "
+                      f"width ({layers} layer runs, batch {B}, prompt {T})", "unit": "tokens/s", "n_gpus": 1,
+            "impl": "b200", "dtype": "bf16", "data": "synthetic (random weights, uniform random token ids)",
+            "higher_is_better": True, "value": sizes["width_2048"]["vipovik"]["decode_tokens_per_s"], "sizes": sizes,
+            "kernels": vipovik_kernels(torch, ops, pk), "clocks": clocks, "peaks": pk}
+    print(json.dumps(line))
+    return 0
+
+
+def vipovik_kernels(torch, ops, pk):
+    """Microseconds of the kernels the design added or changed, alone, at the layer sizes of width 2,048, with the bytes
+    each has to move over its time as a fraction of the measured copy bandwidth, each beside the like kernel of another
+    model."""
+    bf = torch.bfloat16
+    out = {}
+    timed = graph_timer(torch, pk, out)
+    W, H, D, R = 2048, 32, 64, 64                  # time mixing of width 2,048: 32 heads of 64
+    RH, RD, RV = 8, 128, 256                       # retention of that width
+    nh, nkv, hd = 16, 4, 128                       # attention of that width
+    HD = H * D
+    freqs = (10000.0 ** (-2.0 * torch.arange(hd // 2, dtype=torch.float64) / hd)).float().cuda()
+    for rows, segs, tag in ((2048, 1, "prefill_2048"), (8, 8, "decode_8"), (64, 64, "decode_64")):
+        per = rows // segs
+        seg_slot = torch.arange(segs, dtype=torch.int32, device="cuda")
+        cu = torch.arange(0, rows + 1, per, dtype=torch.int32, device="cuda")
+        row_seq = torch.arange(segs, dtype=torch.int32, device="cuda").repeat_interleave(per).contiguous()
+        pos = (torch.arange(rows, dtype=torch.int32, device="cuda") % per) + (1024 if segs > 1 else 0)
+        copies = 4 if segs < 64 else 8
+
+        def mixing():
+            x = (torch.randn(rows, 4 * HD, device="cuda") * 0.5).to(bf)
+            raw, w0, u = torch.randn(rows, HD, device="cuda"), torch.full((HD,), -4.0, device="cuda"), torch.randn(HD, device="cuda")
+            st = torch.zeros(segs, HD * D + W, device="cuda")
+            y = torch.empty(rows, HD, device="cuda")
+            return lambda: ops.time_mixing(x, 0, HD, 2 * HD, raw, w0, u, st, seg_slot, cu, segs, H, D, y, max_seg_rows=per,
+                                           piece_rows=None if pieces else 0)
+        for pieces in ((True, False) if segs == 1 else (True,)):
+            timed(mixing, rows * HD * (3 * 2 + 4 + 4) + 2 * segs * HD * D * 4, f"time_mixing_{tag}" if pieces else f"time_mixing_in_one_piece_{tag}",
+                  copies=copies)
+        # an update and a product per state element and token, three multiply-adds of 32-bit
+        if segs == 1:
+            out[f"time_mixing_{tag}"]["tflops_f32"] = round(6.0 * rows * HD * D / out[f"time_mixing_{tag}"]["us"] / 1e6, 2)
+
+        def retention():
+            qkv = (torch.randn(rows, 2 * RH * RD + 2 * RH * RV, device="cuda") * 0.5).to(bf)
+            om = torch.tensor([2.0 ** (-5 - h) for h in range(RH)], device="cuda")
+            st = torch.zeros(segs, RH * RD * RV, device="cuda")
+            y = torch.empty(rows, RH * RV, device="cuda")
+            dp = ops.retention_piece_decays((1.0 - om.double()).tolist()).cuda()
+            return lambda: ops.retention(qkv, 0, RH * RD, 2 * RH * RD, pos, freqs, RD, RD ** -0.5, om, st, seg_slot, cu, segs, RH, RD, RV,
+                                         y, max_seg_rows=per, piece_decays=dp)
+        timed(retention, rows * ((2 * RH * RD + RH * RV) * 2 + RH * RV * 4) + 2 * segs * RH * RD * RV * 4, f"closest_model_retention_{tag}", copies=copies)
+        if segs == 1:
+            name = f"closest_model_retention_{tag}"
+            out[name]["tflops_f32"] = round(6.0 * rows * RH * RD * RV / out[name]["us"] / 1e6, 2)
+
+        def shift():
+            h = torch.randn(rows, W, device="cuda").to(bf)
+            st = torch.zeros(segs, HD * D + W, device="cuda")
+            mu = torch.rand(5, W, device="cuda")
+            o = torch.empty(rows, 5 * W, dtype=bf, device="cuda")
+            return lambda: ops.token_shift(h, st[:, HD * D:], seg_slot, row_seq, cu, mu, o)
+        timed(shift, rows * W * 6 * 2 + 5 * W * 4 + 2 * segs * W * 4, f"token_shift_{tag}")
+
+        def conv():             # the like kernel: a short convolution over the rows, with the rows before in a state
+            x = torch.randn(rows, 2 * W, device="cuda").to(bf)
+            w, b = torch.randn(2 * W, 4, device="cuda"), torch.zeros(2 * W, device="cuda")
+            st = torch.zeros(segs, 3 * 2 * W, device="cuda")
+            o = torch.empty(rows, 2 * W, dtype=bf, device="cuda")
+            return lambda: ops.causal_conv_act(x, 0, 2 * W, w, b, st, seg_slot, cu, segs, per, "silu", o, update_state=segs > 1)
+        timed(conv, rows * 2 * W * 2 * 2 + 2 * W * 5 * 4 + (2 if segs > 1 else 1) * segs * 3 * 2 * W * 4, f"closest_model_causal_conv_{tag}")
+
+        def blends():
+            x = torch.randn(rows, 5 * W, device="cuda").to(bf)
+            w = (torch.randn(4 * HD + R, W, device="cuda") * 0.02).to(bf)
+            return lambda: ops.linear_blends(x, w, 4, HD, "tanh")
+        fl = 2.0 * rows * (4 * HD + R) * W
+        timed(blends, ((4 * HD + R) * W + rows * (5 * W + 4 * HD)) * 2, f"linear_blends_{tag}", flops=fl)
+
+        def one_product():
+            x = torch.randn(rows, W, device="cuda").to(bf)
+            w = (torch.randn(4 * HD + R, W, device="cuda") * 0.02).to(bf)
+            return lambda: ops.linear(x, w, None)
+        timed(one_product, ((4 * HD + R) * W + rows * (W + 4 * HD)) * 2, f"closest_model_one_product_of_that_size_{tag}", flops=fl)
+
+        def narrow():           # the decays' second matrix: 32-bit sums
+            x = torch.randn(rows, R, device="cuda").to(bf)
+            w = (torch.randn(HD, R, device="cuda") * 0.02).to(bf)
+            return lambda: ops.linear(x, w, None, None, out_dtype=torch.float32)
+        timed(narrow, (HD * R + rows * R) * 2 + rows * HD * 4, f"decay_second_product_{tag}", flops=2.0 * rows * HD * R)
+
+        dq, dk = nh * hd, nkv * hd
+
+        def turn():
+            buf = torch.randn(rows, dq + 2 * dk, device="cuda").to(bf)
+            return lambda: ops.qk_turn_norm(buf, 0, nh, dq, nkv, hd, 1e-6, pos, freqs, hd, 1.2)
+        timed(turn, rows * 2 * (dq + dk) * 2, f"qk_turn_norm_{tag}")
+
+        def prepare():          # Vatevik's: one norm over all of q and one over all of k, then the rotation
+            buf = torch.randn(rows, dq + 2 * dk, device="cuda").to(bf)
+            qw, kw = torch.ones(dq, device="cuda"), torch.ones(dk, device="cuda")
+            return lambda: ops.qk_prepare(buf, 0, nh, dq, nkv, hd, qw, kw, 1e-6, pos, freqs, hd)
+        timed(prepare, rows * 2 * (dq + dk) * 2, f"closest_model_qk_prepare_{tag}")
+
+    # attention of 16 query heads over 4 key/value heads of 128 over a prompt of 2,048 and for 8 decoding rows behind 2,047
+    # keys, a window of 1,024; pages of 16
+    ps, ctx_len, window = 16, 2048, 1024
+    pages = ctx_len // ps
+    bt1 = torch.arange(pages, dtype=torch.int32, device="cuda").view(1, pages)
+    cu1 = torch.tensor([0, ctx_len], dtype=torch.int32, device="cuda")
+    zero1 = torch.zeros(1, dtype=torch.int32, device="cuda")
+
+    def pairs(w):
+        return sum(min(p + 1, w) if w else p + 1 for p in range(ctx_len))
+
+    def prefill(kernel, w, **kw):
+        def make():
+            q = torch.randn(ctx_len, nh * hd, device="cuda").to(bf)
+            k, v = (torch.randn(pages, nkv, ps, hd, device="cuda").to(bf) for _ in range(2))
+            o = torch.empty(ctx_len, nh * hd, dtype=bf, device="cuda")
+            return lambda: kernel(q, k, v, bt1, cu1, zero1, o, 0, 1, ctx_len, nh, nkv, hd, ps, hd ** -0.5, w, **kw)
+        return make
+    nbytes = ctx_len * (2 * nh + 2 * nkv) * hd * 2
+    for w, tag in ((window, "window_1024"), (0, "all_keys")):
+        flops = 4.0 * pairs(w) * nh * hd
+        extra = dict(cap=50.0, keep=16 if w else 0)
+        timed(prefill(ops.paged_prefill_tc5, w, **extra), nbytes, f"attention_prefill_2048_capped_{tag}", flops=flops)
+        timed(prefill(ops.paged_prefill_tc5, w, cap=2.0, keep=16 if w else 0), nbytes, f"attention_prefill_2048_cap_below_the_scores_{tag}", flops=flops)
+        timed(prefill(ops.paged_prefill_tc5, w), nbytes, f"closest_model_attention_prefill_2048_plain_{tag}", flops=flops)
+        timed(prefill(ops.paged_prefill_bf16, w, **extra), nbytes, f"attention_prefill_2048_capped_mma_sync_tiles_{tag}", flops=flops)
+        timed(prefill(ops.paged_prefill_bf16, w), nbytes, f"closest_model_attention_prefill_2048_mma_sync_tiles_{tag}", flops=flops)
+    B = 8
+    btB = torch.arange(B * pages, dtype=torch.int32, device="cuda").view(B, pages)
+    row_seq = torch.arange(B, dtype=torch.int32, device="cuda")
+    posB = torch.full((B,), ctx_len - 1, dtype=torch.int32, device="cuda")
+    slot_map = (btB[:, -1] * ps + ps - 1).contiguous()
+
+    def decode(w, **kw):
+        def make():
+            qkv = torch.randn(B, (nh + 2 * nkv) * hd, device="cuda").to(bf)
+            k, v = (torch.randn(B * pages, nkv, ps, hd, device="cuda").to(bf) for _ in range(2))
+            o = torch.empty(B, nh * hd, dtype=bf, device="cuda")
+            ns = ops.decode_splits(B, nh, ctx_len)
+            scratch = torch.empty(max(1, ops.decode_scratch_floats(B, nh, hd, ns)), device="cuda")
+            counters = torch.zeros(B * nh, dtype=torch.int32, device="cuda")
+            return lambda: ops.paged_decode_bf16(qkv, nh * hd, (nh + nkv) * hd, k, v, btB, row_seq, posB, slot_map, o, scratch,
+                                                 counters, nh, nkv, hd, ps, hd ** -0.5, w, ns, **kw)
+        return make
+    for w, tag in ((window, "window_1024"), (0, "all_keys")):
+        nbytes = B * (w + 16 if w else ctx_len) * 2 * nkv * hd * 2
+        timed(decode(w, cap=50.0, keep=16 if w else 0), nbytes, f"attention_decode_8_capped_{tag}")
+        timed(decode(w), nbytes, f"closest_model_attention_decode_8_plain_{tag}")
     return out
 
 

@@ -179,7 +179,7 @@ def test_long_decoding(dtype):
     ref, _, close = plain_all(cfgd, w, toks)
     moves = rounding_moves(cfgd, w, toks) if dtype == "bfloat16" else None
     eng = make_engine(cfgd, w, dtype)
-    assert_close(run_cut(eng, toks, [20] + [1] * 280), ref, dtype, "decode", close, moves=moves)
+    assert_close(run_cut(eng, toks, [20] + [1] * 280), ref, dtype, "decode", close, tol32=5e-4, moves=moves)
 
 
 def test_two_scales_and_a_zero():
