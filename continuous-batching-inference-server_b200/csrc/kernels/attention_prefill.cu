@@ -207,16 +207,37 @@ paged_prefill_bf16_kernel(const __nv_bfloat16* q, int q_ld, const __nv_bfloat16*
     const int j0 = kt * PF_BN;
     const bool edge = (j0 + PF_BN - 1 > pos0) || (window != 0 && j0 < first_seen(pos0 + PF_BM - 1, window));
     float mx0 = -INFINITY, mx1 = -INFINITY;
+    if constexpr (EXT) {
+      if (cap_log2e > 0.f) {       // capped scores, divided by the rows' scales: scaled once more below
+        const float to_x0 = sc0 / cap_log2e, to_x1 = sc1 / cap_log2e, back0 = 1.f / to_x0, back1 = 1.f / to_x1;
+        float big = 0.f;
+#pragma unroll
+        for (int nt = 0; nt < PF_BN / 8; ++nt)
+#pragma unroll
+          for (int e = 0; e < 2; ++e) {
+            s[nt][e] *= to_x0;
+            s[nt][2 + e] *= to_x1;
+            big = fmaxf(big, fmaxf(fabsf(s[nt][e]), fabsf(s[nt][2 + e])));
+          }
+        if (__any_sync(0xffffffffu, !(big <= TANH_POLY_MAX))) {
+#pragma unroll
+          for (int nt = 0; nt < PF_BN / 8; ++nt)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) s[nt][e] = tanh_exp(s[nt][e]) * (e < 2 ? back0 : back1);
+        } else {
+#pragma unroll
+          for (int nt = 0; nt < PF_BN / 8; ++nt)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) s[nt][e] = tanh_poly(s[nt][e]) * (e < 2 ? back0 : back1);
+        }
+      }
+    }
 #pragma unroll
     for (int nt = 0; nt < PF_BN / 8; ++nt)
 #pragma unroll
       for (int e = 0; e < 2; ++e) {
         const int j = j0 + nt * 8 + 2 * t + e;
         float a = s[nt][e] * sc0, b2 = s[nt][2 + e] * sc1;
-        if constexpr (EXT) {
-          a = capped_score(a, cap_log2e);
-          b2 = capped_score(b2, cap_log2e);
-        }
         if (rates) {
           const int at = PF_BN - 1 - (j - j0);
           a -= s_bias[at + lr0];

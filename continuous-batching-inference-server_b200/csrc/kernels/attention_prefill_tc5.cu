@@ -169,22 +169,6 @@ __device__ __forceinline__ void tmem_st32(unsigned taddr, const float* v) {
   asm volatile("tcgen05.wait::st.sync.aligned;" ::: "memory");
 }
 
-// x * (polynomial in x^2) = tanh(x) for |x| <= 3/4, from a Chebyshev interpolation of tanh(x) / x in x^2 (sixth
-// coefficient last): relative error below 2e-7.
-constexpr float TANH_POLY_MAX = 0.75f;
-__device__ __forceinline__ float tanh_poly(float x) {
-  const float u = x * x;
-  float r = -0.00472395f;
-  r = fmaf(r, u, 0.01959379f);
-  r = fmaf(r, u, -0.05334982f);
-  r = fmaf(r, u, 0.13325515f);
-  r = fmaf(r, u, -0.33332968f);
-  r = fmaf(r, u, 1.0f);
-  return x * r;
-}
-// 1 - 2 / (e^(2x) + 1): absolute error of a few 1e-7, for any x.
-__device__ __forceinline__ float tanh_exp(float x) { return 1.f - __fdividef(2.f, exp2f(fminf(x * 2.8853900817779268f, 126.f)) + 1.f); }
-
 // The 128 softmax threads (warps 2..5) meet at a barrier of their own.
 __device__ __forceinline__ void softmax_warps_meet() {
   __syncwarp();

@@ -113,6 +113,23 @@ __device__ __forceinline__ int kept_end(int p, int window, int keep) {
 // A cap on the scaled scores, cap * tanh(s / cap); cap 0: none.
 __device__ __forceinline__ float capped_score(float s, float cap) { return cap > 0.f ? cap * tanhf(s / cap) : s; }
 
+// The two forms of tanh that the tiled kernels use, where a tile's scores decide on one for a whole warp:
+// x * (polynomial in x^2) = tanh(x) for |x| <= 3/4, from a Chebyshev interpolation of tanh(x) / x in x^2 (sixth
+// coefficient last): relative error below 2e-7.
+constexpr float TANH_POLY_MAX = 0.75f;
+__device__ __forceinline__ float tanh_poly(float x) {
+  const float u = x * x;
+  float r = -0.00472395f;
+  r = fmaf(r, u, 0.01959379f);
+  r = fmaf(r, u, -0.05334982f);
+  r = fmaf(r, u, 0.13325515f);
+  r = fmaf(r, u, -0.33332968f);
+  r = fmaf(r, u, 1.0f);
+  return x * r;
+}
+// 1 - 2 / (e^(2x) + 1): absolute error of a few 1e-7, for any x.
+__device__ __forceinline__ float tanh_exp(float x) { return 1.f - __fdividef(2.f, exp2f(fminf(x * 2.8853900817779268f, 126.f)) + 1.f); }
+
 __device__ __forceinline__ float to_f32(float v) { return v; }
 __device__ __forceinline__ float to_f32(__nv_bfloat16 v) { return __bfloat162float(v); }
 __device__ __forceinline__ void from_f32(float& dst, float v) { dst = v; }

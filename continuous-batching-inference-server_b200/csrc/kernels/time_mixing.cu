@@ -16,7 +16,8 @@
 // long, 1 in steps of short segments), each spread over L lanes: a lane holds runs of four channels, 4 l + 4 L i on, in
 // registers, so its share of a row staged in shared memory is read 16 bytes at a time without bank conflicts and serves CPT
 // columns.  Rows come through shared memory TC at a time (keys, receptances, 1 - w, the block's slice of values); the next
-// TC rows are on their way from memory, into registers, while these are walked.
+// TC rows are on their way from memory, into registers, while these are walked.  (Packed 32-bit multiply-adds and
+// fetching entries in pairs were tried: no faster where the walk is cut into pieces, 1.4 times slower where it is not.)
 //
 // One long prompt offers heads x columns of parallel work only.  Where a step's states are few and its longest segment is
 // long, segments are cut into pieces of `piece_rows` rows that run side by side, in three launches: every piece but a
@@ -29,7 +30,6 @@ namespace cbis {
 
 constexpr int kMixRows = 16;       // rows of a batch for long segments
 constexpr int kMixRowsShort = 4;   // rows of a batch where no segment of the step is longer (decode steps)
-constexpr int kShiftRows = 8;      // rows a block of token_shift walks
 constexpr int kShiftMost = 8;      // blends token_shift takes
 
 enum { kMixWhole = 0, kMixEnds = 1, kMixFromStarts = 2 };
@@ -39,13 +39,13 @@ struct alignas(sizeof(TT) * V) Run {
   TT e[V];
 };
 
-// grid (runs of kShiftRows rows, blocks of columns); a thread takes V columns of every row of the run, with the blends'
-// weights of these columns in registers.  The thread that meets a segment's first row reads the row kept in the state and
-// then replaces it by the segment's last row: no other thread touches these columns of it.
+// grid (runs of `run` rows, blocks of columns); a thread takes V columns of every row of the run, with the blends' weights of
+// these columns in registers, and asks for the next row while it works on one.  The thread that meets a segment's first row
+// reads the row kept in the state and then replaces it by the segment's last row: no other thread touches these columns of it.
 template <typename TT, int V, int N>
 __global__ void __launch_bounds__(256)
 token_shift_kernel(const TT* h, int ld, float* state, long long slot_stride, const int* seg_slot, const int* row_seq,
-                   const int* cu_rows, const float* __restrict__ mu, int n_mix, TT* out, int out_ld, int width, int rows) {
+                   const int* cu_rows, const float* __restrict__ mu, int n_mix, TT* out, int out_ld, int width, int rows, int run) {
   pdl_trigger();
   const int c = (blockIdx.y * blockDim.x + threadIdx.x) * V;
   if (c >= width) return;
@@ -55,11 +55,14 @@ token_shift_kernel(const TT* h, int ld, float* state, long long slot_stride, con
 #pragma unroll
     for (int k = 0; k < V; ++k) m[s][k] = s < n_mix ? mu[(size_t)s * width + c + k] : 0.f;
   pdl_wait();
-  const int r0 = blockIdx.x * kShiftRows, r1 = min(rows, r0 + kShiftRows);
+  const int r0 = blockIdx.x * run, r1 = min(rows, r0 + run);
   float prev[V];
   int have = -1;                       // the row whose values prev holds
+  Run<TT, V> next = *reinterpret_cast<const Run<TT, V>*>(h + (size_t)r0 * ld + c);
   for (int r = r0; r < r1; ++r) {
     const int seq = row_seq[r];
+    const Run<TT, V> now = next;
+    if (r + 1 < r1) next = *reinterpret_cast<const Run<TT, V>*>(h + (size_t)(r + 1) * ld + c);
     TT* o = out + (size_t)r * out_ld + c;
     if (seq < 0) {                     // a padding row of a fixed-size batch
       Run<TT, V> z;
@@ -68,7 +71,6 @@ token_shift_kernel(const TT* h, int ld, float* state, long long slot_stride, con
       for (int s = 0; s < n_mix; ++s) *reinterpret_cast<Run<TT, V>*>(o + (size_t)s * width) = z;
       continue;
     }
-    const Run<TT, V> now = *reinterpret_cast<const Run<TT, V>*>(h + (size_t)r * ld + c);
     float x[V];
 #pragma unroll
     for (int k = 0; k < V; ++k) x[k] = to_f32(now.e[k]);
@@ -412,11 +414,13 @@ template <typename TT, int V>
 static int launch_token_shift(const void* h, int ld, float* state, long long slot_stride, const int* seg_slot,
                               const int* row_seq, const int* cu_rows, const float* mu, int n_mix, void* out, int out_ld,
                               int width, int rows, cudaStream_t st) {
-  const int cols = (width + V - 1) / V, threads = cols >= 256 ? 256 : (cols >= 128 ? 128 : 64);
-  const dim3 grid((rows + kShiftRows - 1) / kShiftRows, (cols + threads - 1) / threads);
+  // few rows: a row a block, narrow blocks; many: runs of rows, so that the blends' weights are read once per run
+  const int cols = (width + V - 1) / V, run = rows <= 256 ? 1 : 4;
+  const int threads = rows <= 256 ? 64 : (cols >= 256 ? 256 : (cols >= 128 ? 128 : 64));
+  const dim3 grid((rows + run - 1) / run, (cols + threads - 1) / threads);
   auto kern = n_mix <= 5 ? token_shift_kernel<TT, V, 5> : token_shift_kernel<TT, V, kShiftMost>;
   return (int)launch_pdl(kern, grid, dim3(threads), 0, st, (const TT*)h, ld, state, slot_stride, seg_slot, row_seq, cu_rows,
-                         mu, n_mix, (TT*)out, out_ld, width, rows);
+                         mu, n_mix, (TT*)out, out_ld, width, rows, run);
 }
 
 }  // namespace cbis

@@ -1182,6 +1182,25 @@ def linear_blends(x, w_all, n_groups, group_n, tail_act=None):
     return out, linear(x[:, n_groups * K:], w_all[n_all:], None, tail_act)
 
 
+TIME_MIXING_ROUND = 4 * 148      # blocks of the walk that run at a time
+
+
+def time_mixing_piece_rows(longest: int, n_segments: int, heads: int, dim: int, total_rows: int = 0) -> int:
+    """Rows of a piece for a step whose longest segment has ``longest`` rows, 0 where segments stay whole: they are cut where
+    the uncut step has about a block a SM or fewer, into as many pieces as run in one round.  ``total_rows``: as in
+    ``retention_piece_rows``."""
+    n_long = min(n_segments, -(-total_rows // longest)) if total_rows > 0 and longest > 0 else n_segments
+    blocks = max(1, n_long * heads * -(-dim // (64 if dim <= 128 else 32)))
+    if longest < RETENTION_PIECES_FROM or blocks > RETENTION_PIECES_MAX_BLOCKS:
+        return 0
+    want = max(2, TIME_MIXING_ROUND // blocks)
+    rows = max(32, -(-(-(-longest // want)) // 16) * 16)
+    n = -(-longest // rows)
+    if n < 2 or n_segments * n > 65535 or n_segments * n * heads * dim * dim * 4 > RETENTION_PIECES_MAX_BYTES:
+        return 0
+    return rows
+
+
 def time_mixing(x, r_off, k_off, v_off, raw, w0, u, state, seg_slot, cu_rows, n_segments, heads, dim, y, max_seg_rows: int = 0,
                 piece_rows=None):
     """The recurrence o = (S + diag(u) k v^T)^T r, S <- diag(w) S + k v^T, w = exp(-exp(raw + w0)), per head over every
@@ -1190,7 +1209,7 @@ def time_mixing(x, r_off, k_off, v_off, raw, w0, u, state, seg_slot, cu_rows, n_
     ``state``: 32-bit ``[slots, >= heads * dim * dim]``; ``max_seg_rows``: the step's longest segment if known.
 
     A segment's rows are walked in order.  Where the step's longest segment is long and its blocks are few
-    (``retention_piece_rows``: the same walk, the same policy), segments are cut into pieces that run side by side; against
+    (``time_mixing_piece_rows``), segments are cut into pieces that run side by side; against
     the walk in one piece the results differ by rounding only.  ``piece_rows``: a piece size of one's own (a multiple of
     16); 0: never cut."""
     _need_cuda(x, raw, w0, u, state, seg_slot, cu_rows, y)
@@ -1205,7 +1224,7 @@ def time_mixing(x, r_off, k_off, v_off, raw, w0, u, state, seg_slot, cu_rows, n_
     longest = int(max_seg_rows or 0)
     rows = 0
     if piece_rows != 0 and longest > 0:
-        rows = int(piece_rows) if piece_rows is not None else retention_piece_rows(longest, n_segments, heads, dim, dim, total_rows=T)
+        rows = int(piece_rows) if piece_rows is not None else time_mixing_piece_rows(longest, n_segments, heads, dim, total_rows=T)
         assert rows >= 0 and rows % 16 == 0
     n_pieces, starts, products = 1, None, None
     if rows and longest > rows:

@@ -133,7 +133,7 @@ def test_a_long_prompt_beside_decoding_rows_is_cut_into_pieces():
     g = torch.Generator().manual_seed(5)
     H, D, lens = 2, 32, [1, 1, 300]
     T = sum(lens)
-    assert ops.retention_piece_rows(300, 3, H, D, D, total_rows=T) > 0
+    assert ops.time_mixing_piece_rows(300, 3, H, D, total_rows=T) > 0
     x, raw = torch.randn(T, 3 * H * D, generator=g), torch.randn(T, H * D, generator=g)
     w0, u = torch.randn(H * D, generator=g) - 4.0, torch.randn(H * D, generator=g)
     cu = torch.tensor([0, 1, 2, T], dtype=torch.int32, device="cuda")
