@@ -71,6 +71,13 @@ __device__ __forceinline__ void gemm_small_m_body(const __nv_bfloat16* A, int ld
   if constexpr (CLUSTER) rank = (int)cluster_ctarank();
   else ksplit = 1;
   const int n0 = (blockIdx.x / ksplit) * (NT * 8);
+  if constexpr (!LOW8 && MT == 1) {      // row tiles of 16 over the blocks' second index (dispatch_small_m)
+    const int m0 = blockIdx.y * 16;
+    A += (size_t)m0 * lda;
+    C += (size_t)m0 * ldc;
+    M = min(M - m0, 16);
+    if (m0 > 0) next_bytes = 0;          // one row of blocks prefetches
+  }
   if constexpr (GROUP) A += (size_t)(n0 / group_n) * K;      // group_n is a multiple of a block's columns
   const int nkb_all = (K + 31) / 32;
   const int per_rank = (nkb_all + ksplit - 1) / ksplit;
@@ -241,7 +248,7 @@ static int launch_small_m(const void* A, int lda, const void* W, const float* bi
   }
   const int blocks = (N + NT * 8 - 1) / (NT * 8) * ksplit;
   if (ksplit == 1)
-    return (int)launch_pdl(kern, dim3(blocks), dim3(SM_WARPS * 32), smem, st, (const __nv_bfloat16*)A, lda,
+    return (int)launch_pdl(kern, dim3(blocks, !LOW8 && MT == 1 ? (M + 15) / 16 : 1), dim3(SM_WARPS * 32), smem, st, (const __nv_bfloat16*)A, lda,
                            (const __nv_bfloat16*)W, bias, (TO*)C, ldc, M, N, K, act, next_w, next_bytes, 1, accumulate, group_n, act_from);
   // clusters of ksplit blocks along x, launched like the others (programmatic dependent launch)
   cudaLaunchConfig_t cfg = {};
@@ -295,6 +302,9 @@ static int dispatch_small_m(const void* A, int lda, const void* W, const float* 
     if (wide) return launch_small_m<1, 2, 4, false, TO>(A, lda, W, bias, C, ldc, M, N, K, act, next_w, next_bytes, st, accumulate, group_n, act_from);
     return launch_small_m<1, 1, 8, false, TO>(A, lda, W, bias, C, ldc, M, N, K, act, next_w, next_bytes, st, accumulate, group_n, act_from);
   }
+  // few columns: 16-row tiles over more blocks (each reads the weights again, from L2) instead of all rows in a few blocks
+  if (!wide && (N + 7) / 8 * ((M + 15) / 16) <= 148)
+    return launch_small_m<1, 1, 8, false, TO>(A, lda, W, bias, C, ldc, M, N, K, act, next_w, next_bytes, st, accumulate, group_n, act_from);
   if (M <= 32) {
     if (wide) return launch_small_m<2, 2, 2, false, TO>(A, lda, W, bias, C, ldc, M, N, K, act, next_w, next_bytes, st, accumulate, group_n, act_from);
     return launch_small_m<2, 1, 4, false, TO>(A, lda, W, bias, C, ldc, M, N, K, act, next_w, next_bytes, st, accumulate, group_n, act_from);
