@@ -225,7 +225,7 @@ __device__ __forceinline__ void decode_tc_item(const __nv_bfloat16* qkv, int ld,
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
         const int o = (e >> 1) * 8 + 2 * t + (e & 1), j = at + o;
-        s4[u][e] = (g == 0 && (j >= kstart || j < kept) && j0 + o < ke) ? sc[e >> 1][e & 1] * scale : -INFINITY;
+        s4[u][e] = (g == 0 && (j >= kstart || (EXT && j < kept)) && j0 + o < ke) ? sc[e >> 1][e & 1] * scale : -INFINITY;
         if (EXT && s4[u][e] > -INFINITY) s4[u][e] = capped_score(s4[u][e], cap);
         if (BIAS && g == 0) s4[u][e] -= distance_bias(slope, rate, (float)max(pos - j, 0));
         mx = fmaxf(mx, s4[u][e]);

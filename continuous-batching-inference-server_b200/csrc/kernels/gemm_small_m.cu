@@ -55,9 +55,9 @@ __device__ __forceinline__ uint4 ldg_stream(const void* p) {
 // CLUSTER: the kernel is launched in clusters of `ksplit` blocks that share a block's columns and split K.  (A kernel that
 // holds cluster instructions is launched through the cluster scheduler even when it never runs them, which was measured
 // to cost the plain form a third of its speed: the two forms are separate kernels.)
-// GROUP: the output's columns come in groups with columns of A of their own (a form of its own: the parameters would cost the
-// others registers).
-template <int MT, int NT, int UNROLL, bool LOW8, typename TO, bool CLUSTER = false, bool GROUP = false>
+// GROUP: the output's columns come in groups with columns of A of their own.  TILES: row tiles of 16 over the blocks' second
+// index.  (Forms of their own: as run-time choices they cost a decode step of the others up to three per cent.)
+template <int MT, int NT, int UNROLL, bool LOW8, typename TO, bool CLUSTER = false, bool GROUP = false, bool TILES = false>
 __device__ __forceinline__ void gemm_small_m_body(const __nv_bfloat16* A, int lda, const __nv_bfloat16* __restrict__ W,
                                                   const float* __restrict__ bias, TO* __restrict__ C, int ldc, int M,
                                                   int N, int K, int act, const void* next_w,
@@ -71,7 +71,7 @@ __device__ __forceinline__ void gemm_small_m_body(const __nv_bfloat16* A, int ld
   if constexpr (CLUSTER) rank = (int)cluster_ctarank();
   else ksplit = 1;
   const int n0 = (blockIdx.x / ksplit) * (NT * 8);
-  if constexpr (!LOW8 && MT == 1) {      // row tiles of 16 over the blocks' second index (dispatch_small_m)
+  if constexpr (TILES) {
     const int m0 = blockIdx.y * 16;
     A += (size_t)m0 * lda;
     C += (size_t)m0 * ldc;
@@ -210,12 +210,12 @@ __device__ __forceinline__ void gemm_small_m_body(const __nv_bfloat16* A, int ld
 
 // Two entry points over the same body: the compiler's own register choice for the general form (80 registers,
 // three blocks per SM), and a cap of 64 registers for the M <= 8 form so that four blocks fit.
-template <int MT, int NT, int UNROLL, typename TO, bool GROUP>
+template <int MT, int NT, int UNROLL, typename TO, bool GROUP, bool TILES>
 __global__ void __launch_bounds__(SM_WARPS * 32)
 gemm_small_m_kernel(const __nv_bfloat16* A, int lda, const __nv_bfloat16* __restrict__ W,
                     const float* __restrict__ bias, TO* __restrict__ C, int ldc, int M, int N, int K, int act,
                     const void* next_w, unsigned long long next_bytes, int ksplit, int accumulate, int group_n, int act_from) {
-  gemm_small_m_body<MT, NT, UNROLL, false, TO, false, GROUP>(A, lda, W, bias, C, ldc, M, N, K, act, next_w, next_bytes, ksplit, accumulate, group_n, act_from);
+  gemm_small_m_body<MT, NT, UNROLL, false, TO, false, GROUP, TILES>(A, lda, W, bias, C, ldc, M, N, K, act, next_w, next_bytes, ksplit, accumulate, group_n, act_from);
 }
 template <int MT, int NT, int UNROLL, typename TO>
 __global__ void __launch_bounds__(SM_WARPS * 32, 4)
@@ -232,7 +232,7 @@ gemm_small_m_low8_ksplit_kernel(const __nv_bfloat16* A, int lda, const __nv_bflo
   gemm_small_m_body<MT, NT, UNROLL, true, TO, true>(A, lda, W, bias, C, ldc, M, N, K, act, next_w, next_bytes, ksplit, accumulate, group_n, act_from);
 }
 
-template <int MT, int NT, int UNROLL, bool LOW8, typename TO>
+template <int MT, int NT, int UNROLL, bool LOW8, typename TO, bool TILES = false>
 static int launch_small_m(const void* A, int lda, const void* W, const float* bias, void* C, int ldc, int M, int N,
                           int K, int act, const void* next_w, unsigned long long next_bytes, cudaStream_t st, int accumulate,
                           int group_n, int act_from, int ksplit = 1) {
@@ -240,7 +240,7 @@ static int launch_small_m(const void* A, int lda, const void* W, const float* bi
   void (*kern)(const __nv_bfloat16*, int, const __nv_bfloat16*, const float*, TO*, int, int, int, int, int, const void*,
                unsigned long long, int, int, int, int);
   if constexpr (LOW8) kern = ksplit > 1 ? gemm_small_m_low8_ksplit_kernel<MT, NT, UNROLL, TO> : gemm_small_m_low8_kernel<MT, NT, UNROLL, TO>;
-  else kern = group_n > 0 ? gemm_small_m_kernel<MT, NT, UNROLL, TO, true> : gemm_small_m_kernel<MT, NT, UNROLL, TO, false>;
+  else kern = group_n > 0 ? gemm_small_m_kernel<MT, NT, UNROLL, TO, true, TILES> : gemm_small_m_kernel<MT, NT, UNROLL, TO, false, TILES>;
   if (!LOW8 && ksplit > 1) return CBIS_ERR_BAD_SIZE;
   if (smem > 48 * 1024) {
     cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
@@ -248,7 +248,7 @@ static int launch_small_m(const void* A, int lda, const void* W, const float* bi
   }
   const int blocks = (N + NT * 8 - 1) / (NT * 8) * ksplit;
   if (ksplit == 1)
-    return (int)launch_pdl(kern, dim3(blocks, !LOW8 && MT == 1 ? (M + 15) / 16 : 1), dim3(SM_WARPS * 32), smem, st, (const __nv_bfloat16*)A, lda,
+    return (int)launch_pdl(kern, dim3(blocks, TILES ? (M + 15) / 16 : 1), dim3(SM_WARPS * 32), smem, st, (const __nv_bfloat16*)A, lda,
                            (const __nv_bfloat16*)W, bias, (TO*)C, ldc, M, N, K, act, next_w, next_bytes, 1, accumulate, group_n, act_from);
   // clusters of ksplit blocks along x, launched like the others (programmatic dependent launch)
   cudaLaunchConfig_t cfg = {};
@@ -304,7 +304,7 @@ static int dispatch_small_m(const void* A, int lda, const void* W, const float* 
   }
   // few columns: 16-row tiles over more blocks (each reads the weights again, from L2) instead of all rows in a few blocks
   if (!wide && (N + 7) / 8 * ((M + 15) / 16) <= 148)
-    return launch_small_m<1, 1, 8, false, TO>(A, lda, W, bias, C, ldc, M, N, K, act, next_w, next_bytes, st, accumulate, group_n, act_from);
+    return launch_small_m<1, 1, 8, false, TO, true>(A, lda, W, bias, C, ldc, M, N, K, act, next_w, next_bytes, st, accumulate, group_n, act_from);
   if (M <= 32) {
     if (wide) return launch_small_m<2, 2, 2, false, TO>(A, lda, W, bias, C, ldc, M, N, K, act, next_w, next_bytes, st, accumulate, group_n, act_from);
     return launch_small_m<2, 1, 4, false, TO>(A, lda, W, bias, C, ldc, M, N, K, act, next_w, next_bytes, st, accumulate, group_n, act_from);
